@@ -8,6 +8,8 @@ from .sobunex import SobunexConfig
 from . import sobunex as _sobunex
 from .pivavik import PivavikConfig
 from . import pivavik as _pivavik
+from .nomutar import NomutarConfig
+from . import nomutar as _nomutar
 from .registry import (config_class_for, config_from_dict, config_from_model_dir,
                        register_architecture, registered_architectures, unregister_architecture)
 
@@ -16,3 +18,4 @@ register_architecture(_lanizen.ARCHITECTURE, LanizenConfig)
 register_architecture(_gidirax.ARCHITECTURE, GidiraxConfig)
 register_architecture(_sobunex.ARCHITECTURE, SobunexConfig)
 register_architecture(_pivavik.ARCHITECTURE, PivavikConfig)
+register_architecture(_nomutar.ARCHITECTURE, NomutarConfig)

@@ -67,6 +67,9 @@ class ModelSpec:
     # as the embedding's rows and are summed before the last norm; every layer's block must be one that takes streams.
     residual_streams: Optional[int] = None
     embedding_norm: Optional[PartSpec] = None  # a norm the embedding's rows pass before the first layer (32-bit in and out)
+    # what is added to the embedding's rows (a part in the role ``embedding``); what it keeps per sequence is one more entry
+    # behind the schedule's in the list of cache requirements
+    embedding_addition: Optional[PartSpec] = None
     logit_softcap: Optional[float] = None      # the logits become cap tanh(logits / cap), after the scale if there is one
 
     def validate(self):

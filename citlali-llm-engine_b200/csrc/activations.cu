@@ -12,7 +12,7 @@
 //                     times the row's weight for the expert (zero: the expert's activations are zeros and its inputs are
 //                     not read), or, with weight_input, of the activation of gate and up each times that weight (the
 //                     expert applied to its weighted input).  The expert for every row comes last, has a width, run and
-//                     limit of its own and weight 1.
+//                     limit of its own and weight 1, or a weight a row of its own (tail_weights).
 #include "api.h"
 #include "common.cuh"
 
@@ -92,7 +92,7 @@ template <typename TZ, typename TO>
 __global__ void __launch_bounds__(256)
 expert_gate_kernel(const TZ* __restrict__ gu, const float* __restrict__ weights, TO* __restrict__ act, int E, int ff, int run,
                    int kind, float limit, float alpha, int tail_ff, int tail_run, float tail_limit,
-                   const float* __restrict__ bias, int weight_input) {
+                   const float* __restrict__ bias, int weight_input, const float* __restrict__ tail_weights) {
     dependents_may_launch();
     wait_for_predecessor();
     const int row = blockIdx.x;
@@ -116,6 +116,7 @@ expert_gate_kernel(const TZ* __restrict__ gu, const float* __restrict__ weights,
             float g = ldf(in, at), u = ldf(in, at + tail_run);
             if (bias) { g += bias[at]; u += bias[at + tail_run]; }
             r = gated(g, u, kind, tail_limit, alpha);
+            if (tail_weights) r *= tail_weights[row];
         }
         stf(o, i, r);
     }
@@ -154,7 +155,8 @@ extern "C" int citlali_add_row_bias(float* y, const float* bias, int rows, int n
 
 extern "C" int citlali_expert_gate(const void* gate_up, int in_dtype, const float* weights, void* act, int act_dtype, int rows,
                                    int E, int ff, int run, int kind, float limit, float alpha, int tail_ff, int tail_run,
-                                   float tail_limit, const float* bias, int weight_input, cudaStream_t stream) {
+                                   float tail_limit, const float* bias, int weight_input, const float* tail_weights,
+                                   cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (E < 0 || ff < 0 || tail_ff < 0 || (E > 0 && (ff <= 0 || run <= 0 || ff % run != 0 || weights == nullptr)) ||
         (tail_ff > 0 && (tail_run <= 0 || tail_ff % tail_run != 0)) || kind < 0 || kind > 2 || E * ff + tail_ff <= 0) {
@@ -168,7 +170,8 @@ extern "C" int citlali_expert_gate(const void* gate_up, int in_dtype, const floa
     return CITLALI_DISPATCH_FLOAT(in_dtype, TZ, [&] {
         return CITLALI_DISPATCH_FLOAT(act_dtype, TO, [&] {
             launch_kernel(expert_gate_kernel<TZ, TO>, grid, 256, 0, stream, (const TZ*)gate_up, weights, (TO*)act, E, ff,
-                          run > 0 ? run : 1, kind, limit, alpha, tail_ff, tail_run > 0 ? tail_run : 1, tail_limit, bias, weight_input);
+                          run > 0 ? run : 1, kind, limit, alpha, tail_ff, tail_run > 0 ? tail_run : 1, tail_limit, bias, weight_input,
+                          tail_weights);
             return CITLALI_LAUNCH_CHECK();
         });
     });

@@ -23,6 +23,14 @@ int citlali_embed_rows(const void* table, int table_dtype, const int32_t* tokens
 int citlali_embed_rows_copies(const void* table, int table_dtype, const int32_t* tokens, float* out, int rows, int hidden,
                               int vocab, float scale, int32_t* error_flag, int copies, size_t copy_stride, cudaStream_t stream);
 
+// The same for one buffer, plus a row of a second table [buckets + 1, hidden] times pair_scale: row (previous token * mul_prev +
+// token * mul_cur) mod buckets, and row `buckets` for a sequence's first token.  state [slots] int32 keeps every sequence's
+// last token between steps (read only past position 0).
+int citlali_embed_rows_paired(const void* table, const void* pairs, int table_dtype, const int32_t* tokens,
+                              const int32_t* row_slot, const int32_t* row_pos, const int32_t* seq_start, int sequences,
+                              int32_t* state, float* out, int rows, int hidden, int vocab, int buckets, long long mul_prev,
+                              long long mul_cur, float scale, float pair_scale, int32_t* error_flag, cudaStream_t stream);
+
 // rows_out = bfloat16(x) [rows, hidden] and sumsq[r, g] = sum of x[r, 32 g .. 32 g + 31]^2 (hidden a multiple of 32):
 // what citlali_gemm_tc_normed's `scale_sumsq` reads, for rows that did not come out of an emitting product.
 int citlali_norm_inputs(const float* x, void* rows_out, float* sumsq, int rows, int hidden, cudaStream_t stream);
@@ -37,6 +45,17 @@ int citlali_concat_rows(const float* a, const float* b, void* out, int out_dtype
 // out[r, :] = x[idx[r], :] * rsqrt(mean(x^2) + eps) * gain   (idx may be null: identity).
 int citlali_rms_norm(const float* x, const void* gain, int gain_dtype, const int32_t* row_index,
                      void* out, int out_dtype, int rows, int hidden, float eps, cudaStream_t stream);
+
+// The same with a row cut into `groups` equal consecutive parts, each divided by its own root mean square.
+int citlali_group_rms_norm(const float* x, const void* gain, int gain_dtype, const int32_t* row_index, void* out, int out_dtype,
+                           int rows, int hidden, int groups, float eps, cudaStream_t stream);
+// h_out[r] = that norm of x[r] and c_out[r] = h + conv(h), conv(h)_t = sum_j taps_w[:, j] h_(t - taps + 1 + j) per channel over
+// a sequence's tokens; state [slot][taps - 1, hidden] float32 keeps a sequence's last rows h, oldest first.  single_tokens:
+// every sequence of the step brings one token (no second kernel is needed to keep them).
+int citlali_group_norm_conv(const float* x, const void* gain, int gain_dtype, const float* taps_w, int taps, float* state,
+                            size_t state_stride, const int32_t* row_slot, const int32_t* seq_start, const int32_t* seq_slot,
+                            int sequences, void* h_out, void* c_out, int out_dtype, int rows, int hidden, int groups, float eps,
+                            int single_tokens, cudaStream_t stream);
 
 // act[m, i] = silu(gate) * up, gate/up taken from one [rows, 2*inter] matrix whose columns
 // alternate in runs of `run`: gate run, up run, gate run, ...
@@ -96,8 +115,13 @@ int citlali_attention_prefill(const void* q, int q_stride, const void* k_pool, c
                               const int32_t* page_table, int page_table_stride,
                               const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
                               void* out, int out_stride, int sequences, int max_new,
-                              int nq, int nkv, int head_dim, int page_size, int window, int keep_first, float scale,
-                              float softcap, const float* gate, size_t gate_stride, cudaStream_t stream);
+                              int nq, int nkv, int head_dim, int value_dim, int page_size, int window, int keep_first,
+                              float scale, float softcap, const float* gate, size_t gate_stride, const float* sink,
+                              const float* turns, int turn_pairs, cudaStream_t stream);
+// sink [nq] (may be null): the softmax's denominator also counts exp(sink[head]), neither scaled nor capped.  turns
+// [rows, value_dim / 2] (cos, sin) (may be null; 16-byte aligned): the result's pairs (m, m + value_dim / 2), or with
+// turn_pairs (2m, 2m + 1), are turned back by the row's angles, ahead of the gate.  Keys and values of different sizes:
+int citlali_attention_prefill_supports_sizes(int head_dim, int value_dim, int page_size);
 
 // The same on tcgen05 (scores and output in tensor memory), for head size 128 and pages of 64.
 // total_rows: rows of q over all sequences; pool_pages: pages of the layer's key and value pools.
@@ -278,15 +302,29 @@ int citlali_attention_window(const void* q, int q_dtype, const void* k_pool, con
                              const int32_t* page_table, int table_stride, const int32_t* row_slot, const int32_t* row_pos,
                              void* out, int rows, int nq, int nkv, int d, int vd, int page_size, int window, int keep_first,
                              int max_keys, float scale, float softcap, const float* gate, size_t gate_stride,
-                             cudaStream_t stream);
+                             const float* sink, const float* turns, int turn_pairs, cudaStream_t stream);
+// (sink, turns, turn_pairs: as citlali_attention_prefill takes them)
+
+// What attention without a convolution reads, from proj [rows, proj_stride] = q (nq d) | k (nkv d) | v (nkv vd) | ...: bias
+// (may be null), an RMS norm over all of q and over all of k with weights of those sizes (may both be null), the rotation of
+// the first rot_dims elements of a head (halves, or with rot_pairs neighbours) with cos and sin times amplitude, and with
+// v_freq [vd / 2] that of the whole value head (halves, or neighbours with v_pairs), whose cos and sin also go to turns
+// [rows, vd / 2].  q to q_out [rows, nq d], k and v to the row's place in the pools.
+int citlali_heads_prepare(const float* proj, int proj_stride, const float* bias, const float* q_gain, const float* k_gain,
+                          float eps, const float* inv_freq, int rot_dims, int rot_pairs, float amplitude, const float* v_freq,
+                          int v_pairs, float* turns, const int32_t* row_slot, const int32_t* row_pos, const int32_t* page_table,
+                          int table_stride, void* k_pool, void* v_pool, int cache_dtype, int page_size, void* q_out, int q_dtype,
+                          int rows, int nq, int nkv, int d, int vd, cudaStream_t stream);
 
 // ---- routed experts ----------------------------------------------------------------------------------------------------
 // weights [rows, E] = softmax(logits) at the `top` best experts among those of the `keep` best of `groups` equal groups of
 // neighbours (a group's score is its largest score; groups <= 1: no groups), 0 elsewhere; chosen [rows, top] (may be
 // null) their indices, best first.
-// The chosen experts' weights are multiplied by weight_scale.  score_kind 1: the scores are sigmoid(logits), each by itself.
+// The chosen experts' weights are multiplied by weight_scale.  score_kind 1: the scores are sigmoid(logits), each by itself;
+// 2: the logits choose, and the weights are the softmax over the chosen.  Rows of logits are `stride` apart; bias [E] (may be
+// null) is added to them.  extra [rows] (may be null) = sigmoid of the column behind the experts'.
 int citlali_moe_route(const float* logits, float* weights, int32_t* chosen, int rows, int E, int groups, int keep, int top,
-                      float weight_scale, int score_kind, cudaStream_t stream);
+                      float weight_scale, int score_kind, int stride, const float* bias, float* extra, cudaStream_t stream);
 // act [rows, E ff + tail_ff] from gate_up [rows, 2 (E ff + tail_ff)], whose columns are, expert after expert, gate and up
 // alternating in runs of `run` (the last expert, which every row uses with weight 1, in runs of `tail_run`).  kind 0:
 // silu(g) u; kind 1: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).  Routed expert e's
@@ -296,7 +334,8 @@ int citlali_moe_route(const float* logits, float* weights, int32_t* chosen, int 
 // experts without biases that is the expert applied to w times its input.
 int citlali_expert_gate(const void* gate_up, int in_dtype, const float* weights, void* act, int act_dtype, int rows, int E,
                         int ff, int run, int kind, float limit, float alpha, int tail_ff, int tail_run, float tail_limit,
-                        const float* bias, int weight_input, cudaStream_t stream);
+                        const float* bias, int weight_input, const float* tail_weights, cudaStream_t stream);
+// (tail_weights [rows], may be null: the last expert's weight a row instead of 1)
 // out = xielu(z + bias) over [rows, n]: u > 0: ap u^2 + u / 2; u <= 0: an (exp(u) - 1 - u) + u / 2.  bias may be null.
 int citlali_bias_xielu(const void* z, int z_dtype, const float* bias, float ap, float an, void* out, int out_dtype, int rows,
                        int n, cudaStream_t stream);

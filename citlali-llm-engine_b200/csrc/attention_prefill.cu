@@ -14,8 +14,11 @@
 // p, query head j reads key/value head j / (heads / kv_heads).  The reference holds all scores
 // in memory and divides per term; this kernel's order differs from it by rounding only.
 //
-// Two options other designs use: a soft cap c on the scaled scores (s <- c tanh(s / c), float, ahead of the mask and the
-// softmax) and an output gate (the result's element is multiplied by the sigmoid of a float32 number of its own).
+// Options other designs use: a soft cap c on the scaled scores (s <- c tanh(s / c), float, ahead of the mask and the
+// softmax); a sink a head (the softmax's denominator also counts exp(sink), neither scaled nor capped); values that were
+// rotated before they were cached (the result is turned back by the row's own angles, through shared memory); and an output
+// gate (the result's element is multiplied by the sigmoid of a float32 number of its own).  Keys and values may differ in
+// size: the tile is then as wide as the larger one, its unused columns zero.
 //
 // The new tokens' keys and values are already in the cache when this runs, so prompts, and
 // runs of tokens that continue a sequence, are the same case: row r of sequence b sits at
@@ -29,9 +32,10 @@ namespace fa {
 
 constexpr int kTileQ = 64, kTileK = 64, kWarps = 4;
 
-// D: head size, a multiple of 16.  Rows in shared memory are D * 2 + 16 bytes apart, which
-// spreads the eight rows of an ldmatrix over all banks.
-template <int D>
+// D: a tile's width, a multiple of 16.  Rows in shared memory are D * 2 + 16 bytes apart, which
+// spreads the eight rows of an ldmatrix over all banks.  EXACT: keys and values are D elements; otherwise dk and dv of them
+// (multiples of 8, at most D).
+template <int D, bool EXACT>
 __global__ void __launch_bounds__(kWarps * 32)
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                          const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
@@ -40,7 +44,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                          const int32_t* __restrict__ seq_past,
                          __nv_bfloat16* __restrict__ out, int out_stride,
                          int nq, int nkv, int window, int keep_first, float scale_log2, float cap_in, float cap_out,
-                         const float* __restrict__ gate, size_t gate_stride) {
+                         const float* __restrict__ gate, size_t gate_stride, const float* __restrict__ sink,
+                         const float2* __restrict__ turns, int turn_pairs, int dk_arg, int dv_arg) {
+    const int dk = EXACT ? D : dk_arg, dv = EXACT ? D : dv_arg;
     constexpr int kRowBytes = D * 2 + 16;
     constexpr int kTileBytes = kTileK * kRowBytes;
     constexpr int kChunksPerRow = D / 8;                     // 16-byte pieces of a row
@@ -66,10 +72,17 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     for (int c = tid; c < kTileQ * kChunksPerRow; c += kWarps * 32) {
         const int r = c / kChunksPerRow, ch = c % kChunksPerRow;
         const uint32_t dst = s_q + r * kRowBytes + ch * 16;
-        if (q0 + r < n_new) cp_async16(dst, q + (size_t)(row0 + q0 + r) * q_stride + (size_t)head * D + ch * 8);
+        if (q0 + r < n_new && ch * 8 < dk) cp_async16(dst, q + (size_t)(row0 + q0 + r) * q_stride + (size_t)head * dk + ch * 8);
         else *reinterpret_cast<uint4*>(smem + r * kRowBytes + ch * 16) = make_uint4(0, 0, 0, 0);
     }
     cp_async_commit();
+    if constexpr (!EXACT) {                                  // columns no key or value has: zeros, written once
+        for (int c = tid; c < 4 * kTileK * kChunksPerRow; c += kWarps * 32) {
+            const int r = c / kChunksPerRow, ch = c % kChunksPerRow;      // rows of both key tiles, then of both value tiles
+            if (ch * 8 >= (r < 2 * kTileK ? dk : dv))
+                *reinterpret_cast<uint4*>(smem + kTileBytes + r * kRowBytes + ch * 16) = make_uint4(0, 0, 0, 0);
+        }
+    }
 
     // key tiles this block visits: from the first key its first row may see to the last key its last row sees
     const int last_pos = past + min(q0 + kTileQ, n_new) - 1;
@@ -83,12 +96,12 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     auto tile_of = [&](int n) { return n <= kept_hi ? n : tile_lo + (n - kept_hi - 1); };
 
     auto load_tile = [&](int tile, int buf) {
-        const size_t base = ((size_t)pages[tile] * nkv + g) * kTileK * D;
+        const size_t base = ((size_t)pages[tile] * nkv + g) * kTileK;
         for (int c = tid; c < kTileK * kChunksPerRow; c += kWarps * 32) {
             const int r = c / kChunksPerRow, ch = c % kChunksPerRow;
-            const size_t src = base + (size_t)r * D + ch * 8;
-            cp_async16(s_k + buf * kTileBytes + r * kRowBytes + ch * 16, k_pool + src);
-            cp_async16(s_v + buf * kTileBytes + r * kRowBytes + ch * 16, v_pool + src);
+            const uint32_t dst = buf * kTileBytes + r * kRowBytes + ch * 16;
+            if (EXACT || ch * 8 < dk) cp_async16(s_k + dst, k_pool + (base + r) * dk + ch * 8);
+            if (EXACT || ch * 8 < dv) cp_async16(s_v + dst, v_pool + (base + r) * dv + ch * 8);
         }
     };
     load_tile(tile_of(0), 0);
@@ -207,13 +220,56 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if (sink) {                                              // in units of log2, as the maxima are once scaled
+        const float share = sink[head] * 1.4426950408889634f;
+        if (m0 != -INFINITY) l0 += fast_exp2(share - m0 * scale_log2);
+        if (m1 != -INFINITY) l1 += fast_exp2(share - m1 * scale_log2);
+    }
     const float inv0 = l0 > 0.0f ? 1.0f / l0 : 0.0f, inv1 = l1 > 0.0f ? 1.0f / l1 : 0.0f;
     const int r0 = q0 + warp * 16 + (lane >> 2), r1 = r0 + 8;
     const int col = (lane & 3) * 2;
+    if (turns) {
+        // the warp's sixteen rows as float32 over the tiles (nobody reads those any more), then every pair turned back
+        constexpr int kPitch = D + 4;
+        float* stage = reinterpret_cast<float*>(smem) + warp * 16 * kPitch;
+#pragma unroll
+        for (int i = 0; i < D / 8; ++i) {
+            *reinterpret_cast<float2*>(stage + (lane >> 2) * kPitch + i * 8 + col) = make_float2(o[i][0] * inv0, o[i][1] * inv0);
+            *reinterpret_cast<float2*>(stage + ((lane >> 2) + 8) * kPitch + i * 8 + col) = make_float2(o[i][2] * inv1, o[i][3] * inv1);
+        }
+        __syncwarp();
+        const int half = dv / 2;                              // a multiple of four: two neighbouring pairs a lane
+        for (int e = lane; e < 16 * (half / 2); e += 32) {
+            const int r = e / (half / 2), p = e % (half / 2) * 2;
+            if (q0 + warp * 16 + r >= n_new) break;
+            const size_t row = row0 + q0 + warp * 16 + r;
+            const float4 t = *reinterpret_cast<const float4*>(turns + row * half + p);        // cos, sin of pairs p and p + 1
+            const int iu = turn_pairs ? 2 * p : p, iv = turn_pairs ? 2 * p + 2 : p + half;    // first two and last two elements
+            float2 a = *reinterpret_cast<const float2*>(stage + r * kPitch + iu), b = *reinterpret_cast<const float2*>(stage + r * kPitch + iv);
+            if (turn_pairs) {
+                a = make_float2(a.x * t.x + a.y * t.y, a.y * t.x - a.x * t.y);
+                b = make_float2(b.x * t.z + b.y * t.w, b.y * t.z - b.x * t.w);
+            } else {
+                const float2 u = a, v = b;
+                a = make_float2(u.x * t.x + v.x * t.y, u.y * t.z + v.y * t.w);
+                b = make_float2(v.x * t.x - u.x * t.y, v.y * t.z - u.y * t.w);
+            }
+            const size_t c = (size_t)head * dv;
+            if (gate) {
+                const float* g = gate + row * gate_stride + c;
+                a.x *= 1.0f / (1.0f + expf(-g[iu])); a.y *= 1.0f / (1.0f + expf(-g[iu + 1]));
+                b.x *= 1.0f / (1.0f + expf(-g[iv])); b.y *= 1.0f / (1.0f + expf(-g[iv + 1]));
+            }
+            *reinterpret_cast<uint32_t*>(out + row * out_stride + c + iu) = pack_bf16(a.x, a.y);
+            *reinterpret_cast<uint32_t*>(out + row * out_stride + c + iv) = pack_bf16(b.x, b.y);
+        }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
+        if (!EXACT && i * 8 >= dv) break;
         float a0 = o[i][0] * inv0, a1 = o[i][1] * inv0, b0 = o[i][2] * inv1, b1 = o[i][3] * inv1;
-        const size_t c = (size_t)head * D + i * 8 + col;
+        const size_t c = (size_t)head * dv + i * 8 + col;
         if (gate) {
             if (r0 < n_new) {
                 const float2 g = *reinterpret_cast<const float2*>(gate + (size_t)(row0 + r0) * gate_stride + c);
@@ -229,13 +285,14 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     }
 }
 
-template <int D>
+template <int D, bool EXACT>
 static int launch(const void* q, int q_stride, const void* k_pool, const void* v_pool, const int32_t* page_table,
                   int page_table_stride, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
                   void* out, int out_stride, int sequences, int max_new, int nq, int nkv, int window, int keep_first,
-                  float scale, float softcap, const float* gate, size_t gate_stride, cudaStream_t stream) {
+                  float scale, float softcap, const float* gate, size_t gate_stride, const float* sink, const float2* turns,
+                  int turn_pairs, int dk, int dv, cudaStream_t stream) {
     constexpr int smem = 5 * kTileK * (D * 2 + 16);
-    auto kernel = attention_prefill_kernel<D>;
+    auto kernel = attention_prefill_kernel<D, EXACT>;
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -249,7 +306,8 @@ static int launch(const void* q, int q_stride, const void* k_pool, const void* v
                                                  window > 0 ? keep_first : 0,
                                                  softcap > 0.0f ? 1.0f : scale * 1.4426950408889634f,
                                                  softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f,
-                                                 softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f, gate, gate_stride);
+                                                 softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f, gate, gate_stride, sink, turns,
+                                                 turn_pairs, dk, dv);
     return CITLALI_LAUNCH_CHECK();
 }
 
@@ -267,6 +325,12 @@ extern "C" int citlali_attention_prefill_supports(int head_dim, int page_size) {
     }
 }
 
+// 1 if citlali_attention_prefill has a kernel for keys of d and values of vd elements.
+extern "C" int citlali_attention_prefill_supports_sizes(int d, int vd, int page_size) {
+    if (d == vd && citlali_attention_prefill_supports(d, page_size)) return 1;
+    return page_size == fa::kTileK && d > 0 && vd > 0 && d % 8 == 0 && vd % 8 == 0 && d <= 256 && vd <= 256;
+}
+
 // Attention of the new tokens of `sequences` sequences (bfloat16, pages of 64).  Sequence b owns
 // rows seq_start[b] .. seq_start[b+1]-1, at positions seq_past[b] + i of slot seq_slot[b];
 // `max_new` is the largest number of new tokens of any sequence.  window > 0: only the last `window` keys and the
@@ -276,13 +340,13 @@ extern "C" int citlali_attention_prefill(const void* q, int q_stride, const void
                                          const int32_t* page_table, int page_table_stride,
                                          const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
                                          void* out, int out_stride, int sequences, int max_new,
-                                         int nq, int nkv, int head_dim, int page_size, int window, int keep_first,
-                                         float scale, float softcap, const float* gate, size_t gate_stride,
-                                         cudaStream_t stream) {
+                                         int nq, int nkv, int head_dim, int value_dim, int page_size, int window, int keep_first,
+                                         float scale, float softcap, const float* gate, size_t gate_stride, const float* sink,
+                                         const float* turns, int turn_pairs, cudaStream_t stream) {
     if (sequences <= 0 || max_new <= 0) return 0;
-    if (!citlali_attention_prefill_supports(head_dim, page_size)) {
-        set_last_error("attention_prefill: no kernel for head size %d with pages of %d (head sizes 16..128 in steps of 16 "
-                       "and 256, pages of 64)", head_dim, page_size);
+    if (!citlali_attention_prefill_supports_sizes(head_dim, value_dim, page_size)) {
+        set_last_error("attention_prefill: no kernel for keys of %d and values of %d with pages of %d (multiples of 8 up to 256, "
+                       "pages of 64)", head_dim, value_dim, page_size);
         return kBadShape;
     }
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || max_new / fa::kTileQ >= 65535 || sequences > 65535) {
@@ -293,16 +357,32 @@ extern "C" int citlali_attention_prefill(const void* q, int q_stride, const void
         set_last_error("attention_prefill: the gate's rows must be 8-byte aligned (row pitch %zu floats)", gate_stride);
         return kBadAlignment;
     }
-    if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 3u)) {
+    if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 3u) || ((uintptr_t)turns & 15u)) {
         set_last_error("attention_prefill: query rows must be 16-byte aligned (row pitch %d elements)", q_stride);
         return kBadAlignment;
     }
-#define CITLALI_FA(DD) case DD: return fa::launch<DD>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, seq_start, \
-                                                      seq_slot, seq_past, out, out_stride, sequences, max_new, nq, nkv, window, keep_first, scale, softcap, gate, gate_stride, stream)
-    switch (head_dim) {
-        CITLALI_FA(16); CITLALI_FA(32); CITLALI_FA(48); CITLALI_FA(64); CITLALI_FA(80); CITLALI_FA(96); CITLALI_FA(112);
-        CITLALI_FA(128); CITLALI_FA(256);
+#define CITLALI_FA(DD, EX) return fa::launch<DD, EX>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, seq_start, \
+                                                      seq_slot, seq_past, out, out_stride, sequences, max_new, nq, nkv, window, keep_first, scale, \
+                                                      softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, head_dim, value_dim, stream)
+    if (head_dim == value_dim) {
+        switch (head_dim) {
+            case 16: CITLALI_FA(16, true);
+            case 32: CITLALI_FA(32, true);
+            case 48: CITLALI_FA(48, true);
+            case 64: CITLALI_FA(64, true);
+            case 80: CITLALI_FA(80, true);
+            case 96: CITLALI_FA(96, true);
+            case 112: CITLALI_FA(112, true);
+            case 128: CITLALI_FA(128, true);
+            case 256: CITLALI_FA(256, true);
+            default: break;
+        }
     }
+    const int widest = head_dim > value_dim ? head_dim : value_dim;
+    if (widest <= 32) CITLALI_FA(32, false);
+    if (widest <= 64) CITLALI_FA(64, false);
+    if (widest <= 96) CITLALI_FA(96, false);
+    if (widest <= 128) CITLALI_FA(128, false);
+    CITLALI_FA(256, false);
 #undef CITLALI_FA
-    return kBadShape;
 }

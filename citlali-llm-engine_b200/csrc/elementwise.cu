@@ -41,6 +41,47 @@ __global__ void embed_rows_kernel(const TW* __restrict__ table, const int32_t* _
     }
 }
 
+// x = E[token] * scale + P[row] * pair_scale with row = (previous token * mul_prev + token * mul_cur) mod buckets, and row
+// `buckets` for a sequence's first token.  The token before a sequence's first row of the step is what the sequence kept
+// (state[slot], read only past position 0); the block of that row leaves the sequence's last token of the step there.
+template <typename TW>
+__global__ void embed_rows_paired_kernel(const TW* __restrict__ table, const TW* __restrict__ pairs,
+                                         const int32_t* __restrict__ tokens, const int32_t* __restrict__ row_slot,
+                                         const int32_t* __restrict__ row_pos, const int32_t* __restrict__ seq_start, int sequences,
+                                         int32_t* __restrict__ state, float* __restrict__ out, int hidden, int vocab, int buckets,
+                                         long long mul_prev, long long mul_cur, float scale, float pair_scale, int32_t* error_flag) {
+    __shared__ int pair_row;
+    dependents_may_launch();
+    wait_for_predecessor();
+    const int row = blockIdx.x;
+    const int tok = tokens[row];
+    const bool ok = tok >= 0 && tok < vocab;
+    if (threadIdx.x == 0) {
+        if (!ok && error_flag) atomicExch(error_flag, 1);
+        const int slot = row_slot[row];
+        const bool starts = row == 0 || row_slot[row - 1] != slot;
+        int at = buckets;
+        if (row_pos[row] > 0) {
+            const long long prev = starts ? state[slot] : tokens[row - 1];
+            at = (int)((((prev * mul_prev + (long long)tok * mul_cur) % buckets) + buckets) % buckets);
+        }
+        pair_row = at;
+        if (starts) {                                         // the sequence whose rows begin here
+            int lo = 0, hi = sequences;
+            while (hi - lo > 1) {
+                const int mid = (lo + hi) / 2;
+                if (seq_start[mid] <= row) lo = mid; else hi = mid;
+            }
+            state[slot] = tokens[seq_start[lo + 1] - 1];
+        }
+    }
+    __syncthreads();
+    const TW* src = table + (size_t)(ok ? tok : 0) * hidden;
+    const TW* pair = pairs + (size_t)pair_row * hidden;
+    float* dst = out + (size_t)row * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? fmaf(ldf(pair, i), pair_scale, ldf(src, i) * scale) : 0.0f;
+}
+
 // What a layer norm that lives in the products around it needs of rows it has not seen come out of a product: the rows
 // as bfloat16 and the sums of their squares over each 32 consecutive features (see citlali_gemm_tc_normed).  One block a
 // row, one warp a group of 32 features at a time.
@@ -218,6 +259,26 @@ extern "C" int citlali_embed_rows_copies(const void* table, int table_dtype, con
 extern "C" int citlali_embed_rows(const void* table, int table_dtype, const int32_t* tokens, float* out,
                                   int rows, int hidden, int vocab, float scale, int32_t* error_flag, cudaStream_t stream) {
     return citlali_embed_rows_copies(table, table_dtype, tokens, out, rows, hidden, vocab, scale, error_flag, 1, 0, stream);
+}
+
+extern "C" int citlali_embed_rows_paired(const void* table, const void* pairs, int table_dtype, const int32_t* tokens,
+                                         const int32_t* row_slot, const int32_t* row_pos, const int32_t* seq_start, int sequences,
+                                         int32_t* state, float* out, int rows, int hidden, int vocab, int buckets,
+                                         long long mul_prev, long long mul_cur, float scale, float pair_scale,
+                                         int32_t* error_flag, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (buckets <= 0 || sequences <= 0 || mul_prev > (1ll << 31) || mul_cur > (1ll << 31) || mul_prev < -(1ll << 31) ||
+        mul_cur < -(1ll << 31)) {
+        set_last_error("embed_rows_paired: %d buckets, %d sequences, multipliers %lld and %lld (32 bits each)", buckets, sequences,
+                       mul_prev, mul_cur);
+        return kBadShape;
+    }
+    return CITLALI_DISPATCH_FLOAT(table_dtype, TW, [&] {
+        launch_kernel(embed_rows_paired_kernel<TW>, rows, 256, 0, stream, (const TW*)table, (const TW*)pairs, tokens, row_slot,
+                      row_pos, seq_start, sequences, state, out, hidden, vocab, buckets, mul_prev, mul_cur, scale, pair_scale,
+                      error_flag);
+        return CITLALI_LAUNCH_CHECK();
+    });
 }
 
 extern "C" int citlali_norm_inputs(const float* x, void* rows_out, float* sumsq, int rows, int hidden, cudaStream_t stream) {

@@ -1,12 +1,14 @@
 // Routed experts: which experts a token uses and with what weight.
 //
 //   moe_route       one warp a row.  scores = softmax(logits) over all E experts (float32), or with score_kind 1 the sigmoid of
-//                   every logit by itself.  The experts form `groups`
+//                   every logit by itself, or with score_kind 2 the logits as they are, whose weights are the softmax over the
+//                   chosen ones only.  A bias an expert is added to the logits first.  The experts form `groups`
 //                   equal groups of neighbours; a group's score is its largest score, and only experts of the `keep` best
 //                   groups can be chosen (groups <= 1 or keep >= groups: all can).  The `top` largest scores among those are
 //                   chosen (of equal scores the lower index first); their weights are the scores themselves, not
-//                   renormalised.  weights [rows, E] receives the score of a chosen expert and 0 for every other; chosen
-//                   [rows, top] the indices, best first.
+//                   renormalised (score_kind 0 and 1).  weights [rows, E] receives the score of a chosen expert and 0 for every other; chosen
+//                   [rows, top] the indices, best first.  With `extra` the column behind the experts' logits is one more number
+//                   of the row (an expert that every row uses), and extra [rows] receives its sigmoid.
 //   moe_scale       act[r, e, j] *= weights[r, e] over act [rows, E, ff]: after this, one product with every expert's output
 //                   matrix side by side is the weighted sum of the chosen experts' outputs (the others contribute zeros).
 #include "api.h"
@@ -18,24 +20,26 @@ constexpr int kMaxExpertsPerLane = 16;      // E <= 512
 
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, int32_t* __restrict__ chosen, int rows, int E,
-                 int groups, int keep, int top, float weight_scale, int score_kind) {
+                 int groups, int keep, int top, float weight_scale, int score_kind, int stride, const float* __restrict__ bias,
+                 float* __restrict__ extra) {
     dependents_may_launch();
     wait_for_predecessor();
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= rows) return;
-    const float* z = logits + (size_t)row * E;
+    const float* z = logits + (size_t)row * stride;
+    if (extra && lane == 0) extra[row] = 1.0f / (1.0f + expf(-z[E]));
     float s[kMaxExpertsPerLane];
     float m = -INFINITY;
 #pragma unroll
     for (int j = 0; j < kMaxExpertsPerLane; ++j) {
         const int e = lane + 32 * j;
-        s[j] = e < E ? z[e] : -INFINITY;
+        s[j] = e < E ? z[e] + (bias ? bias[e] : 0.0f) : -INFINITY;
         m = fmaxf(m, s[j]);
     }
     if (score_kind == 1) {
 #pragma unroll
         for (int j = 0; j < kMaxExpertsPerLane; ++j) s[j] = lane + 32 * j < E ? 1.0f / (1.0f + expf(-s[j])) : 0.0f;
-    } else {
+    } else if (score_kind == 0) {
         m = warp_max(m);
         float sum = 0.0f;
 #pragma unroll
@@ -121,6 +125,21 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
             if (arg == lane + 32 * j) taken |= 1u << j;
         if (lane == 0 && chosen) chosen[(size_t)row * top + round] = arg;
     }
+    if (score_kind == 2) {                                   // softmax over the chosen logits
+        float best = -INFINITY, sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < kMaxExpertsPerLane; ++j)
+            if (taken >> j & 1u) best = fmaxf(best, s[j]);
+        best = warp_max(best);
+#pragma unroll
+        for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+            s[j] = (taken >> j & 1u) ? expf(s[j] - best) : 0.0f;
+            sum += s[j];
+        }
+        sum = warp_sum(sum);
+#pragma unroll
+        for (int j = 0; j < kMaxExpertsPerLane; ++j) s[j] = s[j] / sum;
+    }
 #pragma unroll
     for (int j = 0; j < kMaxExpertsPerLane; ++j) {
         const int e = lane + 32 * j;
@@ -169,10 +188,15 @@ __global__ void moe_scale_vec_kernel(__nv_bfloat16* __restrict__ act, const floa
 using namespace citlali;
 
 extern "C" int citlali_moe_route(const float* logits, float* weights, int32_t* chosen, int rows, int E, int groups, int keep,
-                                 int top, float weight_scale, int score_kind, cudaStream_t stream) {
+                                 int top, float weight_scale, int score_kind, int stride, const float* bias, float* extra,
+                                 cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (score_kind != 0 && score_kind != 1) {
-        set_last_error("moe_route: score kind %d is neither softmax (0) nor sigmoid (1)", score_kind);
+    if (score_kind < 0 || score_kind > 2) {
+        set_last_error("moe_route: score kind %d is neither softmax (0), sigmoid (1) nor a softmax over the chosen (2)", score_kind);
+        return kBadShape;
+    }
+    if (stride < E + (extra ? 1 : 0)) {
+        set_last_error("moe_route: rows of %d logits hold no %d experts%s", stride, E, extra ? " and one more number" : "");
         return kBadShape;
     }
     if (E <= 0 || E > 32 * kMaxExpertsPerLane || top <= 0 || top > E) {
@@ -184,7 +208,7 @@ extern "C" int citlali_moe_route(const float* logits, float* weights, int32_t* c
         return kBadShape;
     }
     launch_kernel(moe_route_kernel, (rows + 3) / 4, 128, 0, stream, logits, weights, chosen, rows, E, groups, keep, top, weight_scale,
-                  score_kind);
+                  score_kind, stride, bias, extra);
     return CITLALI_LAUNCH_CHECK();
 }
 

@@ -34,7 +34,8 @@ def model_is_graph_safe(model) -> bool:
         for part in block.parts():
             if not getattr(part, "graph_safe", False):
                 return False
-    return True
+    addition = getattr(model, "embedding_addition", None)
+    return addition is None or bool(getattr(addition, "graph_safe", False))
 
 
 class _PinnedRing:

@@ -34,6 +34,8 @@ def _build_layers(spec: ModelSpec):
 def expected_tensors(spec: ModelSpec) -> List[TensorSpec]:
     """Every checkpoint tensor the model reads, in a fixed order.  No device is touched."""
     specs = [TensorSpec(spec.embedding_name, (spec.vocab_size, spec.hidden_size), "matrix")]
+    if spec.embedding_addition is not None:
+        specs.extend(build_part("embedding", spec.embedding_addition).tensor_specs())
     if spec.embedding_norm is not None:
         specs.extend(build_part("norm", spec.embedding_norm).tensor_specs())
     for block in _build_layers(spec):
@@ -51,9 +53,13 @@ def expected_tensors(spec: ModelSpec) -> List[TensorSpec]:
 
 def cache_requirements_of(spec: ModelSpec, layers=None) -> List[object]:
     """Per schedule step: what it keeps (a KVRequirement, a StateRequirement, or None for a step that keeps
-    nothing or reads another step's cache).  No device is touched."""
+    nothing or reads another step's cache).  An addition to the embedding's rows has one more entry behind the schedule's.
+    No device is touched."""
     layers = layers if layers is not None else _build_layers(spec)
-    return [None if step.cache_of is not None else layers[step.layer].cache_requirement() for step in spec.schedule]
+    out = [None if step.cache_of is not None else layers[step.layer].cache_requirement() for step in spec.schedule]
+    if spec.embedding_addition is not None:
+        out.append(build_part("embedding", spec.embedding_addition).cache_requirement())
+    return out
 
 
 class DecoderModel:
@@ -64,6 +70,9 @@ class DecoderModel:
         self.layers = _build_layers(spec)
         self.final_norm = build_part("norm", spec.final_norm)
         self.embedding_norm = build_part("norm", spec.embedding_norm) if spec.embedding_norm is not None else None
+        self.embedding_addition = build_part("embedding", spec.embedding_addition) if spec.embedding_addition is not None else None
+        require(spec.residual_streams is None or self.embedding_addition is None,
+                "an addition to the embedding's rows works on one residual stream")
         self.keeps_embedding_output = any(getattr(block, "needs_embedding_output", False) for block in self.layers)
         require(spec.residual_streams is None or (self.embedding_norm is None and not self.keeps_embedding_output),
                 "a norm on the embedding's rows and blocks that read them again work on one residual stream")
@@ -100,6 +109,8 @@ class DecoderModel:
         self.final_norm.bind(weights, ctx)
         if self.embedding_norm is not None:
             self.embedding_norm.bind(weights, ctx)
+        if self.embedding_addition is not None:
+            self.embedding_addition.bind(weights, ctx)
         tie = spec.tie_head_to_embedding
         if tie is None:
             tie = spec.head_name not in weights      # absent head: reuse the embedding (qwen_model.cpp:71-75)
@@ -127,7 +138,12 @@ class DecoderModel:
         emb_scale = 1.0 if spec.embedding_scale is None else float(spec.embedding_scale)
         if streams is None:
             x = torch.empty((batch.rows, spec.hidden_size), dtype=torch.float32, device=ctx.device)
-            ops.embed_rows(self.embedding, batch.tokens, x, ctx.error_flag, emb_scale)
+            if self.embedding_addition is not None:
+                at = len(spec.schedule)
+                self.embedding_addition.forward(self.embedding, batch, x, cache.view(at) if cache.has_view(at) else None,
+                                                ctx.error_flag, emb_scale)
+            else:
+                ops.embed_rows(self.embedding, batch.tokens, x, ctx.error_flag, emb_scale)
             if self.embedding_norm is not None:
                 x = self.embedding_norm.forward(x, out_dtype=torch.float32)
             # blocks that read the embedding's rows again get them apart from the residual, which the layers change in place

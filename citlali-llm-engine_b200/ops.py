@@ -107,6 +107,22 @@ def embed_rows_streams(table: torch.Tensor, tokens: torch.Tensor, out: torch.Ten
                                            ctypes.c_size_t(rows * hidden), _stream()), "embed_rows")
 
 
+def embed_rows_paired(table, pairs, batch, state, out, error_flag, mul_prev: int, mul_cur: int, scale: float = 1.0,
+                      pair_scale: float = 1.0):
+    """``out = table[token] * scale + pairs[row] * pair_scale``, row = (previous token * mul_prev + token * mul_cur) mod
+    (``pairs``' rows - 1), its last row for a sequence's first token.  ``state`` int32 [slots, 1]: the sequences' last tokens."""
+    _need_cuda(table, pairs, state, out, error_flag)
+    rows, hidden = out.shape
+    require(batch.tokens.dtype == torch.int32 and batch.tokens.numel() == rows and out.dtype == torch.float32
+            and state.dtype == torch.int32 and table.shape[1] == hidden and pairs.shape[1] == hidden and pairs.shape[0] > 1
+            and pairs.dtype == table.dtype, "embed_rows_paired: shapes or dtypes do not fit")
+    _check(lib().citlali_embed_rows_paired(
+        _ptr(table), _ptr(pairs), _i(_dtype_code(table)), _ptr(batch.tokens), _ptr(batch.row_slot), _ptr(batch.row_pos),
+        _ptr(batch.seq_start), _i(batch.sequences), _ptr(state), _ptr(out), _i(rows), _i(hidden), _i(table.shape[0]),
+        _i(pairs.shape[0] - 1), ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), _f(scale), _f(pair_scale),
+        _ptr(error_flag), _stream()), "embed_rows_paired")
+
+
 def scale_(x: torch.Tensor, scale: float):
     """x *= scale in place (float32)."""
     _need_cuda(x)
@@ -143,6 +159,39 @@ def rms_norm(x: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor,
         require(x.shape[0] == rows, "rms_norm: shapes do not fit")
     _check(lib().citlali_rms_norm(_ptr(x), _ptr(gain), _i(_dtype_code(gain)), _ptr(row_index), _ptr(out),
                                   _i(_dtype_code(out)), _i(rows), _i(hidden), _f(eps), _stream()), "rms_norm")
+
+
+def group_rms_norm(x, gain, groups: int, eps: float, out, row_index=None):
+    """``rms_norm`` with a row cut into ``groups`` equal parts, each divided by its own root mean square."""
+    _need_cuda(x, gain, out, row_index)
+    rows, hidden = out.shape
+    require(x.dtype == torch.float32 and x.shape[1] == hidden and gain.numel() == hidden
+            and (x.shape[0] == rows if row_index is None else (row_index.dtype == torch.int32 and row_index.numel() == rows)),
+            "group_rms_norm: shapes or dtypes do not fit")
+    _check(lib().citlali_group_rms_norm(_ptr(x), _ptr(gain), _i(_dtype_code(gain)), _ptr(row_index), _ptr(out),
+                                        _i(_dtype_code(out)), _i(rows), _i(hidden), _i(groups), _f(eps), _stream()),
+           "group_rms_norm")
+
+
+def group_norm_conv(x, gain, groups: int, eps: float, taps_w, state, batch, h_out, c_out):
+    """``h_out`` = :func:`group_rms_norm` of every row, ``c_out`` = h + a causal convolution of h over a sequence's tokens
+    (``taps_w`` float32 [hidden, taps]).  ``state`` float32 [slots, (taps - 1) * hidden]: the sequences' last rows h."""
+    _need_cuda(x, gain, taps_w, state, h_out, c_out)
+    rows, hidden = x.shape
+    taps = taps_w.shape[1]
+    require(x.dtype == torch.float32 and gain.numel() == hidden and taps_w.dtype == torch.float32 and taps_w.shape[0] == hidden
+            and h_out.shape == x.shape and c_out.shape == x.shape and h_out.dtype == c_out.dtype
+            and (taps == 1 or (state is not None and state.dtype == torch.float32 and state.shape[1] == (taps - 1) * hidden)),
+            "group_norm_conv: shapes or dtypes do not fit")
+    single = batch.is_decode
+    _check(lib().citlali_group_norm_conv(
+        _ptr(x), _ptr(gain), _i(_dtype_code(gain)), _ptr(taps_w), _i(taps), _ptr(state),
+        _sz(state.shape[1] if state is not None else 0), _ptr(batch.row_slot), _ptr(batch.seq_start), _ptr(batch.seq_slot),
+        _i(batch.sequences), _ptr(h_out), _ptr(c_out), _i(_dtype_code(h_out)), _i(rows), _i(hidden), _i(groups), _f(eps),
+        _i(1 if single else 0), _stream()), "group_norm_conv" if (single or taps == 1) else "group_norm_conv_kept")
+
+
+_KERNELS_PER_CALL["group_norm_conv_kept"] = 2
 
 
 def swiglu(gate_up: torch.Tensor, act: torch.Tensor, run: int):
@@ -262,20 +311,31 @@ def attention(q, q_stride, cache_view, batch, out, nq, nkv, head_dim, window, sc
 
 
 def attention_prefill(q, q_stride, k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, sequences, max_new,
-                      nq, nkv, head_dim, page_size, window, scale, keep_first=0, softcap=0.0, gate=None):
-    """``softcap`` c > 0: scaled scores become c tanh(s / c).  ``gate``: float32 [rows, heads * head size] (rows may be
-    further apart than they are long), the output is multiplied by its sigmoids."""
-    _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out)
+                      nq, nkv, head_dim, page_size, window, scale, keep_first=0, softcap=0.0, gate=None, value_dim=None,
+                      sink=None, turns=None, turn_pairs=False):
+    """``softcap`` c > 0: scaled scores become c tanh(s / c).  ``gate``: float32 [rows, heads * value size] (rows may be
+    further apart than they are long), the output is multiplied by its sigmoids.  ``value_dim``: a value's size (None: the
+    key's).  ``sink``: float32, a number a head the softmax's denominator counts the exponential of.  ``turns``: float32
+    [rows, value size / 2, 2], the angles the result's pairs are turned back by."""
+    _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, sink, turns)
+    vd = head_dim if value_dim is None else value_dim
+    _check_sink_and_turns(sink, turns, nq, out.shape[0], vd)
     require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
             "attention_prefill: bfloat16 only")
     require(gate is None or (gate.is_cuda and gate.dtype == torch.float32 and gate.stride(1) == 1
-                             and gate.shape == (out.shape[0], nq * head_dim)), "attention_prefill: the gate does not fit")
+                             and gate.shape == (out.shape[0], nq * vd)), "attention_prefill: the gate does not fit")
     _check(lib().citlali_attention_prefill(
         _ptr(q), _i(q_stride), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _i(page_table.shape[1]),
         _ptr(seq_start), _ptr(seq_slot), _ptr(seq_past), _ptr(out), _i(out.shape[1]), _i(sequences), _i(max_new),
-        _i(nq), _i(nkv), _i(head_dim), _i(page_size), _i(window or 0), _i(keep_first or 0), _f(scale),
-        _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _stream()),
-        "attention_prefill")
+        _i(nq), _i(nkv), _i(head_dim), _i(vd), _i(page_size), _i(window or 0), _i(keep_first or 0), _f(scale),
+        _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink), _ptr(turns),
+        _i(1 if turn_pairs else 0), _stream()), "attention_prefill")
+
+
+def _check_sink_and_turns(sink, turns, heads, rows, value_dim):
+    require(sink is None or (sink.dtype == torch.float32 and sink.numel() == heads), "the sinks are float32, a number a head")
+    require(turns is None or (turns.dtype == torch.float32 and turns.numel() == rows * value_dim),
+            "the angles to turn back by are float32 [rows, value size / 2, 2]")
 
 
 def attention_prefill_tc(q, q_stride, k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, sequences, max_new,
@@ -752,29 +812,53 @@ def conv_heads_prepare(proj, taps_w, state, conv_off, q_gain, k_gain, inv_freq, 
         _i(1 if write_cache else 0), _ptr(bias), _stream()), "conv_heads_prepare")
 
 
-def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scale, softcap=0.0, gate=None):
+def heads_prepare(proj, batch, kv, q_out, nq, nkv, d, vd, bias=None, q_gain=None, k_gain=None, eps=0.0, inv_freq=None,
+                  rot_dims=0, rot_pairs=False, amplitude=1.0, v_freq=None, v_pairs=False, turns=None):
+    """Bias, a norm over all of q and over all of k (``q_gain``/``k_gain`` of those sizes), rotations of q and k (``inv_freq``)
+    and of v (``v_freq``; its cosines and sines go to ``turns`` [rows, vd / 2, 2]) and the cache write, in one pass over the
+    projection's rows.  ``proj`` may be wider than q | k | v."""
+    _need_cuda(proj, bias, q_gain, k_gain, inv_freq, v_freq, turns, kv.keys, kv.values, kv.page_table, q_out)
+    rows = proj.shape[0]
+    C = (nq + nkv) * d + nkv * vd
+    f32 = lambda t, n: t is None or (t.dtype == torch.float32 and t.numel() == n)
+    require(proj.dtype == torch.float32 and proj.shape[1] >= C and q_out.shape == (rows, nq * d) and kv.keys.shape[-1] == d
+            and kv.values.shape[-1] == vd and kv.keys.shape[-3] == nkv and kv.keys.dtype == kv.values.dtype and f32(bias, C)
+            and f32(q_gain, nq * d) and f32(k_gain, nkv * d) and (rot_dims == 0 or (inv_freq is not None and f32(inv_freq, rot_dims // 2)))
+            and f32(v_freq, vd // 2) and (v_freq is None or (turns is not None and f32(turns, rows * vd))),
+            "heads_prepare: shapes or dtypes do not fit")
+    _check(lib().citlali_heads_prepare(
+        _ptr(proj), _i(proj.shape[1]), _ptr(bias), _ptr(q_gain), _ptr(k_gain), _f(eps), _ptr(inv_freq), _i(rot_dims),
+        _i(1 if rot_pairs else 0), _f(amplitude), _ptr(v_freq), _i(1 if v_pairs else 0), _ptr(turns), _ptr(batch.row_slot),
+        _ptr(batch.row_pos), _ptr(kv.page_table), _i(kv.page_table.shape[1]), _ptr(kv.keys), _ptr(kv.values),
+        _i(_dtype_code(kv.keys)), _i(kv.page_size), _ptr(q_out), _i(_dtype_code(q_out)), _i(rows), _i(nq), _i(nkv), _i(d), _i(vd),
+        _stream()), "heads_prepare")
+
+
+def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scale, softcap=0.0, gate=None, sink=None,
+                     turns=None, turn_pairs=False):
     """Attention of every row over its slot's cache, through a window that keeps the first tokens.  bfloat16 steps that
-    bring runs of tokens, with keys and values of one size the tensor-core kernel has, run that kernel; steps of single
+    bring runs of tokens, with keys and values of sizes the tensor-core kernel takes, run that kernel; steps of single
     tokens, the 32-bit path and other sizes run the kernel whose launch depends on the row count alone.  ``softcap`` c > 0:
-    the scaled scores become c tanh(s / c).  ``gate``: float32 columns of a matrix (a view whose rows may be further apart
+    the scaled scores become c tanh(s / c).  ``sink``, ``turns``, ``turn_pairs``: see :func:`attention_prefill`.  ``gate``: float32 columns of a matrix (a view whose rows may be further apart
     than they are long), the output is multiplied by their sigmoids element by element."""
-    _need_cuda(q, kv.keys, kv.values, kv.page_table, out)
+    _need_cuda(q, kv.keys, kv.values, kv.page_table, out, sink, turns)
     rows = q.shape[0]
     require(q.shape == (rows, nq * d) and out.shape == (rows, nq * vd) and q.dtype == out.dtype,
             "attention_window: shapes or dtypes do not fit")
+    _check_sink_and_turns(sink, turns, nq, rows, vd)
     gate_stride = 0
     if gate is not None:
         require(gate.is_cuda and gate.dtype == torch.float32 and gate.shape == (rows, nq * vd) and gate.stride(1) == 1,
                 "attention_window: the gate is float32 [rows, heads * value size] with unit column stride")
         gate_stride = gate.stride(0)
     softcap = float(softcap or 0.0)
-    if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and d == vd and not batch.is_decode
+    if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and not batch.is_decode
             and (nq * d) % 8 == 0 and not torch.cuda.is_current_stream_capturing()
             and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 8 == 0))
-            and lib().citlali_attention_prefill_supports(_i(d), _i(kv.page_size))):
+            and lib().citlali_attention_prefill_supports_sizes(_i(d), _i(vd), _i(kv.page_size))):
         attention_prefill(q, nq * d, kv.keys, kv.values, kv.page_table, batch.seq_start, batch.seq_slot, batch.seq_past, out,
                           batch.sequences, batch.max_new, nq, nkv, d, kv.page_size, window, scale, keep_first=keep_first,
-                          softcap=softcap, gate=gate)
+                          softcap=softcap, gate=gate, value_dim=vd, sink=sink, turns=turns, turn_pairs=turn_pairs)
         return
     longest = kv.page_table.shape[1] * kv.page_size          # a bound that no step's lengths change
     max_keys = min(longest, window + keep_first) if window else longest
@@ -782,23 +866,27 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
         _ptr(q), _i(_dtype_code(q)), _ptr(kv.keys), _ptr(kv.values), _i(_dtype_code(kv.keys)), _ptr(kv.page_table),
         _i(kv.page_table.shape[1]), _ptr(batch.row_slot), _ptr(batch.row_pos), _ptr(out), _i(rows), _i(nq), _i(nkv), _i(d),
         _i(vd), _i(kv.page_size), _i(int(window or 0)), _i(int(keep_first or 0)), _i(max_keys), _f(scale), _f(softcap),
-        _ptr(gate), _sz(gate_stride), _stream()), "attention_window")
+        _ptr(gate), _sz(gate_stride), _ptr(sink), _ptr(turns), _i(1 if turn_pairs else 0), _stream()), "attention_window")
 
 
 # ---- routed experts -----------------------------------------------------------------------------------------------
 
-ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 
 
-def moe_route(logits, weights, groups, keep, top, chosen=None, weight_scale=1.0, score="softmax"):
-    _need_cuda(logits, weights, chosen)
+def moe_route(logits, weights, groups, keep, top, chosen=None, weight_scale=1.0, score="softmax", bias=None, extra=None):
+    """``bias``: float32, a number an expert added to the logits.  ``extra`` float32 [rows]: receives the sigmoid of the one
+    column that ``logits`` has behind the experts'."""
+    _need_cuda(logits, weights, chosen, bias, extra)
     require(score in ROUTER_SCORES, f"moe_route: unknown score '{score}'; known: {', '.join(ROUTER_SCORES)}")
-    rows, E = logits.shape
-    require(logits.dtype == torch.float32 and weights.dtype == torch.float32 and weights.shape == logits.shape
-            and (chosen is None or (chosen.dtype == torch.int32 and chosen.shape == (rows, top))),
+    rows, E = weights.shape
+    require(logits.dtype == torch.float32 and weights.dtype == torch.float32
+            and logits.shape == (rows, E if extra is None else E + 1)
+            and (bias is None or (bias.dtype == torch.float32 and bias.numel() == E))
+            and (extra is None or (extra.dtype == torch.float32 and extra.numel() == rows)) and (chosen is None or (chosen.dtype == torch.int32 and chosen.shape == (rows, top))),
             "moe_route: shapes or dtypes do not fit")
     _check(lib().citlali_moe_route(_ptr(logits), _ptr(weights), _ptr(chosen), _i(rows), _i(E), _i(int(groups or 0)),
-                                   _i(int(keep or 0)), _i(top), _f(weight_scale), _i(ROUTER_SCORES[score]), _stream()),
+                                   _i(int(keep or 0)), _i(top), _f(weight_scale), _i(ROUTER_SCORES[score]), _i(logits.shape[1]), _ptr(bias), _ptr(extra), _stream()),
            "moe_route")
 
 
@@ -814,12 +902,15 @@ EXPERT_ACTIVATIONS = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}
 
 
 def expert_gate(gate_up, weights, act, E, ff, run, kind, limit=0.0, alpha=1.0, tail_ff=0, tail_run=1, tail_limit=0.0,
-                bias=None, weight_input=False):
+                bias=None, weight_input=False, tail_weights=None):
     """The gated activation of ``E`` routed experts (times the row's weight for each) and of a last expert that every row
     uses, from one product ``gate_up`` [rows, 2 (E ff + tail_ff)] into ``act`` [rows, E ff + tail_ff].  ``bias``: float32,
     a number a column of ``gate_up``, added first.  ``weight_input``: the row's weight multiplies gate and up ahead of
-    the activation (the expert applied to the weighted input) instead of the activation's result."""
-    _need_cuda(gate_up, weights, act, bias)
+    the activation (the expert applied to the weighted input) instead of the activation's result.  ``tail_weights``: float32
+    [rows], the last expert's weight (None: 1)."""
+    _need_cuda(gate_up, weights, act, bias, tail_weights)
+    require(tail_weights is None or (tail_weights.dtype == torch.float32 and tail_weights.numel() == act.shape[0]),
+            "expert_gate: the last expert's weights do not fit")
     require(bias is None or (bias.dtype == torch.float32 and bias.numel() == gate_up.shape[1]), "expert_gate: the bias does not fit")
     rows = act.shape[0]
     n = E * ff + tail_ff
@@ -829,7 +920,7 @@ def expert_gate(gate_up, weights, act, E, ff, run, kind, limit=0.0, alpha=1.0, t
     _check(lib().citlali_expert_gate(_ptr(gate_up), _i(_dtype_code(gate_up)), _ptr(weights), _ptr(act), _i(_dtype_code(act)),
                                      _i(rows), _i(E), _i(ff), _i(run), _i(EXPERT_ACTIVATIONS[kind]), _f(limit), _f(alpha),
                                      _i(tail_ff), _i(tail_run), _f(tail_limit), _ptr(bias), _i(1 if weight_input else 0),
-                                     _stream()), "expert_gate")
+                                     _ptr(tail_weights), _stream()), "expert_gate")
 
 
 def bias_xielu(z, bias, ap, an, out):

@@ -22,3 +22,7 @@ from . import sigmoid_attention   # one more built-in mixer
 from .block import SandwichNormBlock
 from .feed_forward import XieluFeedForward
 from .sigmoid_attention import SigmoidAttention
+from . import embedding, mixer_input   # what is added to embedding rows, what mixers read
+from .embedding import HashedPairEmbedding
+from .mixer_input import ResidualConv
+from .norm import GroupedRMSNorm

@@ -19,6 +19,8 @@ Interfaces (all tensors are on the model's device; ``x`` is the float32 residual
   position order, ``batch.row_slot`` / ``batch.row_pos`` say whose they are and where.
 * feed-forward: ``forward(h, batch, residual)`` adds its output into ``residual`` in place.
 * position encoding: ``__init__(params, head_dim)``; see :mod:`.rotary`.
+* mixer input: what a mixer reads instead of the normed rows; see :mod:`.mixer_input`.
+* embedding: what is added to a token's embedding row; see :mod:`.embedding`.
 * block: ``__init__(layer_spec)`` builds the parts it knows by name from ``layer_spec.parts``
   (:func:`build_part`); ``parts()``, ``tensor_specs()``, ``cache_requirement()``, ``bind``;
   ``forward(x, batch, cache_view, write_cache)`` updates ``x`` in place.
@@ -33,7 +35,7 @@ import torch
 from ..errors import require
 
 _REGISTRIES: Dict[str, Dict[str, type]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {},
+    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "mixer_input": {}, "embedding": {},
 }
 
 

@@ -229,7 +229,9 @@ class SandwichNormBlock:
 
 class ParallelResidualBlock:
     """h = norm(x); x += mixer(h) + feed_forward(h): one norm, and both sub-layers read what it gives.  Parts by name:
-    ``norm``, ``mixer``, ``feed_forward`` (either sub-layer may be absent).  Both outputs are added into the float32
+    ``norm``, ``mixer``, ``feed_forward`` (either sub-layer may be absent), and optionally ``mixer_input``: the mixer then
+    reads what that part makes of the normed rows (the layer's cache is the pair of the two parts'), the feed-forward the
+    normed rows as they are.  Both outputs are added into the float32
     residual by the products that end the sub-layers (32-bit additions)."""
 
     def __init__(self, layer_spec):
@@ -237,14 +239,17 @@ class ParallelResidualBlock:
         self.norm = build_part("norm", layer_spec.part("norm"))
         self.mixer = build_part("mixer", layer_spec.part("mixer")) if has("mixer") else None
         self.feed_forward = build_part("feed_forward", layer_spec.part("feed_forward")) if has("feed_forward") else None
+        self.mixer_input = build_part("mixer_input", layer_spec.part("mixer_input")) if has("mixer_input") and has("mixer") else None
 
     def parts(self):
-        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+        return [p for p in (self.norm, self.mixer_input, self.mixer, self.feed_forward) if p is not None]
 
     def tensor_specs(self):
         return [t for p in self.parts() for t in p.tensor_specs()]
 
     def cache_requirement(self):
+        if self.mixer_input is not None:
+            return (self.mixer.cache_requirement(), self.mixer_input.cache_requirement())
         return self.mixer.cache_requirement() if self.mixer is not None else None
 
     def bind(self, weights, ctx):
@@ -255,9 +260,14 @@ class ParallelResidualBlock:
         return self.norm
 
     def forward(self, x, batch, cache_view, write_cache=True):
-        h = self.norm.forward(x)
-        if self.mixer is not None:
-            self.mixer.forward(h, batch, cache_view, x, write_cache)
+        if self.mixer_input is not None:
+            mixer_view, input_view = cache_view
+            h, m = self.mixer_input.forward(self.norm, x, batch, input_view)
+            self.mixer.forward(m, batch, mixer_view, x, write_cache)
+        else:
+            h = self.norm.forward(x)
+            if self.mixer is not None:
+                self.mixer.forward(h, batch, cache_view, x, write_cache)
         if self.feed_forward is not None:
             self.feed_forward.forward(h, batch, x)
         return x

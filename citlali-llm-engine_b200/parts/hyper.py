@@ -44,7 +44,7 @@ class HyperConnectionBlock:
             if not has(role):
                 continue
             norm = build_part("norm", layer_spec.part(norm_name))
-            require(isinstance(norm, RMSNorm), f"the norm in front of a {role} on several streams must be an RMS norm")
+            require(type(norm) is RMSNorm, f"the norm in front of a {role} on several streams must be an RMS norm over the whole row")
             part = build_part(role, layer_spec.part(role))
             for k in ("in", "out", "mix"):
                 require(f"{role}_{k}" in names, f"a layer on several streams needs the tensor name '{role}_{k}'")

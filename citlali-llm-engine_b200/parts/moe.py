@@ -1,7 +1,8 @@
 """Routed experts: a feed-forward made of ``experts`` small gated feed-forwards of which every token uses ``top``.
 
 Router logits z = W_router h in 32-bit; scores s = softmax(z) over all experts (``score`` "sigmoid": s = sigmoid(z), every
-expert's score by itself).  The experts form ``groups`` equal groups of
+expert's score by itself; "softmax_chosen": the logits choose, and the weights are the softmax over the chosen logits
+only).  With ``router_bias`` a number an expert is added to the logits.  The experts form ``groups`` equal groups of
 neighbours; a group's score is the largest score in it, and only experts of the ``keep_groups`` best groups can be chosen
 (``groups`` None: no groups).  The ``top`` experts with the largest scores among those are chosen; their weights are their
 scores times ``weight_scale``, not renormalised.  An expert is  W_down act(W_gate h, W_up h), without biases; the output is
@@ -12,8 +13,9 @@ times h (the weight then meets gate and up ahead of the activation: act(w W_gate
 * ``clamped_swish``: g' = min(g, limit), u' = clamp(u, -limit, limit); act = g' sigmoid(alpha g') (u' + 1), with ``limit``
   and ``alpha`` (default 1.702) from the parameters.
 
-``shared``: {"intermediate_size", "limit"} of one more expert of the same form that runs for every row and is added with
-weight 1; its matrices ride in the same two products, behind the routed experts'.
+``shared``: {"intermediate_size", "limit", "weight"} of one more expert of the same form that runs for every row and is added
+with weight 1, or with ``weight`` "sigmoid" times sigmoid(w h), one number a row from a vector w that rides in the router's
+product; its matrices ride in the same two products, behind the routed experts'.
 
 How it runs: the router is a product with a float32 result; one kernel turns a row's logits into a row of weights (zero
 for an expert that was not chosen); the experts' gate and up matrices are ONE product for all experts (the gate in its
@@ -23,8 +25,9 @@ by side are ONE product that sums over experts.  Nothing depends on counts known
 only, so a decoding step replays as a graph; the price is that every expert's matrices are applied to every row.
 
 Parameters: hidden_size, experts, top, intermediate_size, groups, keep_groups, weight_scale, score, weight_on, activation,
-limit, alpha, shared; ``names``: {"router": name, "gate": [names], "up": [names], "down": [names], "shared": {"gate", "up", "down"}}
-(default ``<prefix>.router``, ``<prefix>.e<i>.{gate,up,down}`` and ``<prefix>.shared.{gate,up,down}``).
+limit, alpha, shared, router_bias; ``names``: {"router": name, "router_bias": name, "gate": [names], "up": [names], "down":
+[names], "shared": {"gate", "up", "down", "weight"}} (default ``<prefix>.router``, ``<prefix>.router.b``,
+``<prefix>.e<i>.{gate,up,down}``, ``<prefix>.shared.{gate,up,down}`` and ``<prefix>.shared.sg``).
 """
 from __future__ import annotations
 
@@ -32,7 +35,8 @@ import torch
 
 from .. import ops
 from ..errors import require
-from .base import register_part
+from ..weights.loader import TensorSpec
+from .base import bind_vector, register_part
 from .linear import DenseLinear, ExpertDown, ExpertGateUp
 
 
@@ -67,6 +71,9 @@ class RoutedExperts:
         shared = params.get("shared")
         self.shared_ff, self.shared_limit = 0, 0.0
         gate_up_tail = down_tail = None
+        self.shared_weighted, router_names, router_sizes = False, [str(n.get("router") or f"{prefix}.router")], [self.E]
+        self.router_bias_name = str(n.get("router_bias") or f"{prefix}.router.b") if params.get("router_bias") else None
+        self.router_bias = None
         if shared is not None:
             self.shared_ff = int(shared["intermediate_size"])
             self.shared_limit = float(shared.get("limit") or 0.0)
@@ -76,7 +83,12 @@ class RoutedExperts:
             name = lambda role: str(sn.get(role) or f"{prefix}.shared.{role}")
             gate_up_tail = (name("gate"), name("up"), self.shared_ff)
             down_tail = (name("down"), self.shared_ff)
-        self.router = DenseLinear([str(n.get("router") or f"{prefix}.router")], [self.E], self.hidden)
+            require(shared.get("weight") in (None, "sigmoid"), f"{prefix}: the weight of the expert for every row is 'sigmoid' or None")
+            self.shared_weighted = shared.get("weight") is not None
+            if self.shared_weighted:
+                router_names.append(str(sn.get("weight") or f"{prefix}.shared.sg"))
+                router_sizes.append(1)
+        self.router = DenseLinear(router_names, router_sizes, self.hidden)
         self.gate_up = ExpertGateUp(each("gate"), each("up"), self.ff, self.hidden, tail=gate_up_tail)
         self.down = ExpertDown(each("down"), self.ff, self.hidden, tail=down_tail)
         self.prefix = prefix
@@ -84,23 +96,32 @@ class RoutedExperts:
         self.plain = self.activation == "silu" and shared is None and not self.weight_input
 
     def tensor_specs(self):
-        return self.router.tensor_specs() + self.gate_up.tensor_specs() + self.down.tensor_specs()
+        bias = [TensorSpec(self.router_bias_name, (self.E,), "state")] if self.router_bias_name is not None else []
+        return self.router.tensor_specs() + bias + self.gate_up.tensor_specs() + self.down.tensor_specs()
 
     def bind(self, weights, ctx):
         self.router.bind(weights, ctx)
         self.gate_up.bind(weights, ctx)
         self.down.bind(weights, ctx)
+        if self.router_bias_name is not None:
+            self.router_bias = bind_vector(weights, self.router_bias_name, self.E, ctx)
         self.dtype = ctx.dtype
 
     def route(self, h):
         """The row's weights for every expert, float32 [rows, experts]: its score where chosen, zero elsewhere."""
+        return self._route(h)[0]
+
+    def _route(self, h):
+        """The weights, and the weight of the expert for every row, float32 [rows] (None: 1)."""
         logits = self.router.forward(h, out_dtype=torch.float32)
-        weights = torch.empty_like(logits)
-        ops.moe_route(logits, weights, self.groups, self.keep, self.top, weight_scale=self.weight_scale, score=self.score)
-        return weights
+        weights = torch.empty((h.shape[0], self.E), dtype=torch.float32, device=h.device)
+        extra = torch.empty((h.shape[0],), dtype=torch.float32, device=h.device) if self.shared_weighted else None
+        ops.moe_route(logits, weights, self.groups, self.keep, self.top, weight_scale=self.weight_scale, score=self.score,
+                      bias=self.router_bias, extra=extra)
+        return weights, extra
 
     def forward(self, h, batch, residual, overwrite=False):
-        weights = self.route(h)
+        weights, extra = self._route(h)
         if self.plain:
             act = self.gate_up.forward_gated(h, self.gate_up.run)
             if act is None:
@@ -111,7 +132,8 @@ class RoutedExperts:
             gu = self.gate_up.forward(h, out_dtype=torch.float32)
             act = torch.empty((h.shape[0], self.E * self.ff + self.shared_ff), dtype=self.dtype, device=h.device)
             ops.expert_gate(gu, weights, act, self.E, self.ff, self.gate_up.run, self.activation, self.limit, self.alpha,
-                            self.shared_ff, self.gate_up.tail_run, self.shared_limit, weight_input=self.weight_input)
+                            self.shared_ff, self.gate_up.tail_run, self.shared_limit, weight_input=self.weight_input,
+                            tail_weights=extra)
         if overwrite:
             self.down.forward(act, out=residual)
         else:

@@ -11,6 +11,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..errors import require
 from ..weights.loader import TensorSpec
 from .base import bind_gain, bind_vector, register_part
 
@@ -35,6 +36,10 @@ class RMSNorm:
             self.gain = (self.gain.to(torch.float32) + self.offset).contiguous()
         self.dtype = ctx.dtype
 
+    def group_terms(self):
+        """(gain, parts of a row that are normed one by one, eps): for a kernel that runs this norm itself."""
+        return self.gain, 1, self.eps
+
     def gain_moves_downstream(self) -> torch.Tensor:
         """The part behind this norm has multiplied its weights by the gain: from now on the norm only divides by the
         root mean square (its kernel gets a gain of ones).  Returns the gain."""
@@ -49,6 +54,26 @@ class RMSNorm:
         rows = x.shape[0] if row_index is None else row_index.numel()
         out = torch.empty((rows, self.size), dtype=out_dtype or self.dtype, device=x.device)
         ops.rms_norm(x, self.gain, self.eps, out, row_index)
+        return out
+
+
+class GroupedRMSNorm(RMSNorm):
+    """An RMS norm over ``groups`` equal consecutive parts of the row: every part is divided by its own
+    sqrt(mean(part^2) + eps), then the whole row is multiplied by the gain (``offset + w``, as in :class:`RMSNorm`)."""
+
+    def __init__(self, params, prefix: str):
+        super().__init__(params, prefix)
+        self.groups = int(params["groups"])
+        require(self.groups >= 1 and self.size % self.groups == 0,
+                f"{prefix}: a row of {self.size} does not split into {self.groups} equal parts")
+
+    def group_terms(self):
+        return self.gain, self.groups, self.eps
+
+    def forward(self, x: torch.Tensor, row_index=None, out_dtype=None) -> torch.Tensor:
+        rows = x.shape[0] if row_index is None else row_index.numel()
+        out = torch.empty((rows, self.size), dtype=out_dtype or self.dtype, device=x.device)
+        ops.group_rms_norm(x, self.gain, self.groups, self.eps, out, row_index)
         return out
 
 
@@ -102,4 +127,5 @@ class LayerNorm:
 
 
 register_part("norm", "rms_norm", RMSNorm)
+register_part("norm", "grouped_rms_norm", GroupedRMSNorm)
 register_part("norm", "layer_norm", LayerNorm)

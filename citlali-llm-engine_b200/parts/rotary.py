@@ -19,10 +19,51 @@ keys are stored; ``batch.row_pos`` holds each row's position.  An encoding with 
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..errors import require
 from .base import register_part
+
+
+def rotation_table(dims: int, base: float, scaling=None):
+    """(float32 frequencies [dims / 2], amplitude) of a rotation of ``dims`` elements: f_i = base^(-2i / dims), computed in
+    double and rounded once, and what cosine and sine are multiplied by.  ``scaling`` (None: none) stretches them for longer
+    sequences:
+
+    * ``{"kind": "wavelength", "factor", "low", "high", "original"}`` (as published with Llama 3.1): with the wavelength l =
+      2 pi / f, f stays where l < original / high, becomes f / factor where l > original / low, and is blended between;
+    * ``{"kind": "ramp", "factor", "original", "fast", "slow"}`` (YaRN): with d(t) = dims ln(original / (2 pi t)) / (2 ln
+      base), a ramp over i from floor(d(fast)) to ceil(d(slow)) goes from f to f / factor; cosine and sine are multiplied by
+      0.1 ln(factor) + 1.
+    """
+    f = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
+    amplitude = 1.0
+    if scaling is not None:
+        kind, factor, original = scaling["kind"], float(scaling["factor"]), float(scaling["original"])
+        if kind == "wavelength":
+            low, high = float(scaling["low"]), float(scaling["high"])
+
+            def stretched(v):
+                l = 2.0 * math.pi / v
+                if l < original / high:
+                    return v
+                if l > original / low:
+                    return v / factor
+                keep = (original / l - low) / (high - low)
+                return (1.0 - keep) * v / factor + keep * v
+            f = [stretched(v) for v in f]
+        elif kind == "ramp":
+            at = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+            lo = max(math.floor(at(float(scaling["fast"]))), 0)
+            hi = min(math.ceil(at(float(scaling["slow"]))), dims - 1)
+            ramp = lambda i: min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            f = [v / factor * ramp(i) + v * (1.0 - ramp(i)) for i, v in enumerate(f)]
+            amplitude = 0.1 * math.log(factor) + 1.0
+        else:
+            require(False, f"unknown scaling of a rotation '{kind}'; known: wavelength, ramp")
+    return torch.tensor(f, dtype=torch.float64).to(torch.float32), amplitude
 
 
 class RotaryHalfSplit:

@@ -5,20 +5,27 @@ For a token with input h:  q (``heads`` of ``dim``), k (``kv_heads`` of ``dim``)
 projections of h, without biases unless ``biases`` says otherwise (a bias a channel, added to what the convolution gives;
 with no convolution: to the projection); each channel then passes a causal convolution over time (``conv`` taps, no bias, zeros before
 the sequence's start; None: none).  q and k heads pass an RMS norm over ``dim`` with a weight shared by the heads
-(``qk_norm_eps`` None: none), then the rotation of the first ``rot_dims`` elements of a head in neighbouring pairs
-(2i, 2i+1) by position * ``rot_base``^(-2i/rot_dims); the rest of a head, and v, pass unchanged.  Query head j reads key
+(``qk_norm_eps`` None: none; ``qk_norm_over`` "projection": over all of q and over all of k at once, ahead of the split into
+heads, with weights of those sizes), then the rotation of the first ``rot_dims`` elements of a head in neighbouring pairs
+(2i, 2i+1), or with ``rot_layout`` "halves" in pairs (i, i + rot_dims/2), by position * ``rot_base``^(-2i/rot_dims), the
+frequencies stretched by ``rot_scaling`` (see :func:`~.rotary.rotation_table`) if given; the rest of a head passes unchanged,
+and so does v, unless ``value_rot_base`` b is given: then v is rotated over its whole length, pair m by position *
+b^(-2m/vdim), before it is cached, and a head's output is turned back by the same angles of the row's own position (ahead of
+the gate), so that a value is seen rotated by its distance.  Query head j reads key
 head j // (heads / kv_heads).  Position p sees key j if j <= p and (p - j < ``window`` or j < ``keep_first``); ``window``
 None: every earlier key.  Kept tokens keep their own positions.  Scores times ``scale``, then with ``softcap`` c the
-score s becomes c tanh(s / c); an ordinary softmax over the visible keys, the weighted sum of values; with ``gate``
+score s becomes c tanh(s / c); a softmax over the visible keys (``sink``: its denominator also counts exp(z), with z a
+learned number a head ("heads") or the given number; z is not scaled, not capped, and has no value), the weighted sum of values; with ``gate``
 "elements" the heads side by side are multiplied element by element by sigmoid(W_g h), a projection of the same input
 without a bias that rides in the q | k | v product; then the output matrix.
 
-The convolution, head norm, rotation and the cache write are one kernel; scores and softmax are float32.  The cache holds
+The convolution (or the norms over the whole projections), head norm, rotations and the cache write are one kernel; scores and softmax are float32.  The cache holds
 keys and values in pages (``KVRequirement`` with the window and the kept tokens: pages that hold neither are given back);
 beside it a sequence keeps the last ``conv - 1`` projected rows in a float32 region, so the mixer asks for two caches.
 
 Parameters: hidden_size, heads, kv_heads, dim, vdim, conv, qk_norm_eps, rot_dims, rot_base, scale, window, keep_first,
-softcap, biases, gate; ``names``: full tensor names by role (q, k, v, q_conv, k_conv, v_conv, q_norm, k_norm, o, gate,
+softcap, biases, gate, qk_norm_over, rot_layout, rot_scaling, value_rot_base, value_rot_layout (default: rot_layout), sink;
+``names``: full tensor names by role (q, k, v, q_conv, k_conv, v_conv, q_norm, k_norm, o, gate, sink,
 q_bias, k_bias, v_bias; the biases default to the matrix's name with ``.b``, the gate to ``<prefix>.g``).
 """
 from __future__ import annotations
@@ -32,8 +39,10 @@ from ..weights.loader import TensorSpec
 from .base import bind_vector, register_part
 from .delta import bind_float32
 from .linear import DenseLinear
+from .rotary import rotation_table
 
-_ROLES = ("q", "k", "v", "q_conv", "k_conv", "v_conv", "q_norm", "k_norm", "o")
+_ROLES = ("q", "k", "v", "q_conv", "k_conv", "v_conv", "q_norm", "k_norm", "o", "sink")
+_LAYOUTS = ("pairs", "halves")
 
 
 class WindowAttention:
@@ -58,6 +67,22 @@ class WindowAttention:
         self.has_gate = params.get("gate") is not None
         require(params.get("gate") in (None, "elements"), f"{prefix}: gate must be 'elements' or None")
         require(self.softcap >= 0.0, f"{prefix}: softcap must be positive or None")
+        self.norm_whole = {"head": False, "projection": True}.get(str(params.get("qk_norm_over") or "head"))
+        require(self.norm_whole is not None, f"{prefix}: qk_norm_over must be 'head' or 'projection'")
+        self.rot_layout = str(params.get("rot_layout") or "pairs")
+        self.rot_scaling = params.get("rot_scaling")
+        self.v_base = None if params.get("value_rot_base") is None else float(params["value_rot_base"])
+        self.v_layout = str(params.get("value_rot_layout") or self.rot_layout)
+        require(self.rot_layout in _LAYOUTS and self.v_layout in _LAYOUTS, f"{prefix}: a rotation's layout is 'pairs' or 'halves'")
+        require(self.v_base is None or self.vd % 2 == 0, f"{prefix}: rotated values need an even size, not {self.vd}")
+        self.sink = params.get("sink")
+        require(self.sink is None or self.sink == "heads" or isinstance(self.sink, (int, float)),
+                f"{prefix}: sink must be 'heads', a number or None")
+        # one kernel prepares heads behind a convolution or with a norm a head, another everything else
+        self.plain_heads = not self.has_conv and (self.eps is None or self.norm_whole)
+        require(self.plain_heads or (not self.norm_whole and self.rot_layout == "pairs" and self.v_base is None
+                                     and (self.rot_scaling is None or self.rot_scaling["kind"] != "ramp")),
+                f"{prefix}: a convolution or a norm a head goes with the 'pairs' rotation of q and k only")
         require(self.nq % self.nkv == 0, f"{prefix}: {self.nq} query heads are not a multiple of {self.nkv} key/value heads")
         require(self.rot_dims % 2 == 0 and self.rot_dims <= self.d,
                 f"{prefix}: {self.rot_dims} rotated elements must be even and at most the head size {self.d}")
@@ -84,10 +109,15 @@ class WindowAttention:
                       TensorSpec(nm["k_conv"], (self.nkv * self.d, self.taps), "state"),
                       TensorSpec(nm["v_conv"], (self.nkv * self.vd, self.taps), "state")]
         if self.eps is not None:
-            specs += [TensorSpec(nm["q_norm"], (self.d,), "gain"), TensorSpec(nm["k_norm"], (self.d,), "gain")]
+            specs += [TensorSpec(nm["q_norm"], (self.norm_sizes()[0],), "gain"), TensorSpec(nm["k_norm"], (self.norm_sizes()[1],), "gain")]
+        if self.sink == "heads":
+            specs.append(TensorSpec(nm["sink"], (self.nq,), "state"))
         if self.has_biases:
             specs += [TensorSpec(nm[r + "_bias"], (size,), "state") for r, size in zip(("q", "k", "v"), self.sizes)]
         return specs
+
+    def norm_sizes(self):
+        return (self.nq * self.d, self.nkv * self.d) if self.norm_whole else (self.d, self.d)
 
     def cache_requirement(self):
         kv = KVRequirement(self.nkv, self.d, self.window, value_dim=self.vd, keep_first=self.keep_first)
@@ -107,15 +137,20 @@ class WindowAttention:
             self.conv_w = torch.ones((self.C, 1), dtype=torch.float32, device=ctx.device)
         self.q_gain = self.k_gain = None
         if self.eps is not None:
-            self.q_gain = bind_float32(weights, nm["q_norm"], (self.d,), ctx)
-            self.k_gain = bind_float32(weights, nm["k_norm"], (self.d,), ctx)
+            self.q_gain = bind_float32(weights, nm["q_norm"], (self.norm_sizes()[0],), ctx)
+            self.k_gain = bind_float32(weights, nm["k_norm"], (self.norm_sizes()[1],), ctx)
         self.bias = None
         if self.has_biases:
             self.bias = torch.cat([bind_vector(weights, nm[r + "_bias"], size, ctx)
                                    for r, size in zip(("q", "k", "v"), self.sizes)]).contiguous()
-        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-        self.inv_freq = (torch.pow(torch.tensor(self.rot_base, dtype=torch.float64), -2.0 * i / max(self.rot_dims, 1))
-                         .to(torch.float32).to(ctx.device))
+        freq, self.amplitude = rotation_table(self.rot_dims, self.rot_base, self.rot_scaling)
+        self.inv_freq = freq.to(ctx.device)
+        self.v_freq = None if self.v_base is None else rotation_table(self.vd, self.v_base)[0].to(ctx.device)
+        self.sinks = None
+        if self.sink == "heads":
+            self.sinks = bind_vector(weights, nm["sink"], self.nq, ctx)
+        elif self.sink is not None:
+            self.sinks = torch.full((self.nq,), float(self.sink), dtype=torch.float32, device=ctx.device)
         self.dtype = ctx.dtype
 
     def forward(self, h, batch, cache_view, residual, write_cache=True, overwrite=False):
@@ -127,13 +162,23 @@ class WindowAttention:
         rows = batch.rows
         proj = self.qkv.forward(h, out_dtype=torch.float32)
         q = torch.empty((rows, self.nq * self.d), dtype=self.dtype, device=proj.device)
-        ops.conv_heads_prepare(proj, self.conv_w, state, 0, self.q_gain, self.k_gain, self.inv_freq, self.rot_dims, batch, kv,
-                               q, self.nq, self.nkv, self.d, self.vd, float(self.eps or 0.0), bias=self.bias)
+        turns = None
+        if self.plain_heads:
+            if self.v_freq is not None:
+                turns = torch.empty((rows, self.vd // 2, 2), dtype=torch.float32, device=proj.device)
+            ops.heads_prepare(proj, batch, kv, q, self.nq, self.nkv, self.d, self.vd, bias=self.bias, q_gain=self.q_gain,
+                              k_gain=self.k_gain, eps=float(self.eps or 0.0), inv_freq=self.inv_freq, rot_dims=self.rot_dims,
+                              rot_pairs=self.rot_layout == "pairs", amplitude=self.amplitude, v_freq=self.v_freq,
+                              v_pairs=self.v_layout == "pairs", turns=turns)
+        else:
+            ops.conv_heads_prepare(proj, self.conv_w, state, 0, self.q_gain, self.k_gain, self.inv_freq, self.rot_dims, batch, kv,
+                                   q, self.nq, self.nkv, self.d, self.vd, float(self.eps or 0.0), bias=self.bias)
         if self.taps > 1:
             ops.conv_keep(proj, proj.shape[1], self.taps, self.C, state, 0, batch)
         out = torch.empty((rows, self.nq * self.vd), dtype=self.dtype, device=proj.device)
         ops.attention_window(q, kv, batch, out, self.nq, self.nkv, self.d, self.vd, self.window, self.keep_first, self.scale,
-                             softcap=self.softcap, gate=proj[:, self.C:] if self.has_gate else None)
+                             softcap=self.softcap, gate=proj[:, self.C:] if self.has_gate else None, sink=self.sinks,
+                             turns=turns, turn_pairs=self.v_layout == "pairs")
         if overwrite:
             self.o.forward(out, out=residual)
         else:
