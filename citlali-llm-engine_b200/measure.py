@@ -4,7 +4,8 @@ Used by ``bench.py --design lanizen`` (beside the Qwen3 dense decoder), ``--desi
 closest design the library has: both mix delta-rule layers with windowed attention) and ``--design sobunex`` (beside
 Gidirax: both have windowed attention with key and value sizes of their own, layer norms on the sub-layers' outputs and
 experts whose weights are not renormalised) and ``--design pivavik`` (beside Sobunex: both are made of attention layers
-only, with windows, output gates, biases, and dense and routed feed-forwards in turn).  A size is a width and a number of layers; both models get that width, that
+only, with windows, output gates, biases, and dense and routed feed-forwards in turn) and ``--design nomutar`` (beside
+Pivavik: both run mixer and feed-forward side by side on one norm and have windowed attention with a soft cap).  A size is a width and a number of layers; both models get that width, that
 many layers, feed-forwards of equal parameter count (8 width^2: two matrices of 4 width, or three of 8/3 width) and
 the same vocabulary, with random weights in bfloat16.  Measured per model: one prompt in one step (tokens a second),
 one decode step of ``batch`` sequences at ``context`` through the session's ``decode`` (the replayed graph where the
@@ -102,6 +103,28 @@ def pivavik_config(width: int, layers: int, vocab: int, window: int = 1024):
     if layers >= 3:
         d["loop"] = {"start": 1, "stop": layers - 1, "times": 1}
     return config_from_dict(d)
+
+
+def nomutar_config(width: int, layers: int, vocab: int, window: int = 1024):
+    """The three attention layers in turn (the second kind twice in four), heads of 128, four query heads a key/value head;
+    dense feed-forwards of 8/3 width and sixteen experts of which a token uses four, plus one of the same size for every token
+    (about 8 width^2 parameters in all experts of a layer); four parts in the norm, a convolution of four taps."""
+    heads = max(1, width // 128)
+    ff = max(64, (width // 6 + 32) // 64 * 64)
+    dense = {"kind": "dense", "ff": (8 * width // 3 + 255) // 256 * 256}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 16, "top": 4}, "shared": {"ff": ff}}
+    sizes = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    first = dict(sizes, softcap=50.0, mask={"size": window}, rot={"base": 500000.0, "dims": 64, "scaling": {
+        "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})
+    second = dict(sizes, softcap=30.0, mask={"size": window}, rot={"base": 10000.0, "dims": 128, "scaling": {
+        "factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 4096}})
+    third = dict(sizes, rot={"base": 10000.0, "dims": 128})
+    order = [("attention", first, dense), ("attention_2", second, moe), ("attention_3", third, moe), ("attention_2", second, dense)]
+    return config_from_dict({
+        "architecture": "Nomutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5, "groups": 4}, "residual_mult": 0.5,
+        "embedding": {"scale": 2.0, "bigram": {"buckets": 32749, "mul_prev": 1021, "mul_cur": 31}}, "canon": {"taps": 4},
+        "logit_softcap": 30.0,
+        "layers": [{"type": t, "mixer": dict(m), "mlp": dict(f)} for t, m, f in (order[i % 4] for i in range(layers))]})
 
 
 def qwen3_config(width: int, layers: int, vocab: int):
@@ -233,7 +256,7 @@ def measure_model(config, prompt_tokens: int, batch: int, context: int, steps: i
 
 
 DESIGNS = {"lanizen": (lanizen_config, "qwen3"), "gidirax": (gidirax_config, "lanizen"), "sobunex": (sobunex_config, "gidirax"),
-           "pivavik": (pivavik_config, "sobunex"), "qwen3": (qwen3_config, None)}
+           "pivavik": (pivavik_config, "sobunex"), "nomutar": (nomutar_config, "pivavik"), "qwen3": (qwen3_config, None)}
 
 
 def run(design: str, sizes, prompt_tokens: int, batch: int, context: int, steps: int, warmup: int) -> dict:
