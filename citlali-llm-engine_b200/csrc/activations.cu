@@ -122,6 +122,42 @@ expert_gate_kernel(const TZ* __restrict__ gu, const float* __restrict__ weights,
     }
 }
 
+// The same with four neighbouring columns a thread (widths and runs that are multiples of four, 16-byte rows): a piece lies
+// within one run of one expert.
+template <typename TZ, typename TO>
+__global__ void __launch_bounds__(256)
+expert_gate_vec_kernel(const TZ* __restrict__ gu, const float* __restrict__ weights, TO* __restrict__ act, int E, int ff, int run,
+                       int kind, float limit, float alpha, int tail_ff, int tail_run, float tail_limit,
+                       const float* __restrict__ bias, int weight_input, const float* __restrict__ tail_weights) {
+    dependents_may_launch();
+    wait_for_predecessor();
+    const int row = blockIdx.x;
+    const int routed = E * ff, n = routed + tail_ff;
+    const TZ* in = gu + (size_t)row * 2 * n;
+    TO* o = act + (size_t)row * n;
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4; i < n; i += gridDim.y * blockDim.x * 4) {
+        const bool tail = i >= routed;
+        const int e = tail ? 0 : i / ff, j = tail ? i - routed : i - e * ff, rn = tail ? tail_run : run;
+        const float w = tail ? (tail_weights ? tail_weights[row] : 1.0f) : weights[(size_t)row * E + e];
+        float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (tail || w != 0.0f) {
+            const int blk = j / rn;
+            const size_t at = (size_t)2 * (i - j) + (size_t)blk * 2 * rn + (j - blk * rn);
+            float4 g = load4(in + at), u = load4(in + at + rn);
+            if (bias) {
+                const float4 bg = *reinterpret_cast<const float4*>(bias + at), bu = *reinterpret_cast<const float4*>(bias + at + rn);
+                g.x += bg.x; g.y += bg.y; g.z += bg.z; g.w += bg.w;
+                u.x += bu.x; u.y += bu.y; u.z += bu.z; u.w += bu.w;
+            }
+            const bool inside = weight_input && !tail;
+            const float wi = inside ? w : 1.0f, wo = inside ? 1.0f : w, lim = tail ? tail_limit : limit;
+            r = make_float4(wo * gated(wi * g.x, wi * u.x, kind, lim, alpha), wo * gated(wi * g.y, wi * u.y, kind, lim, alpha),
+                            wo * gated(wi * g.z, wi * u.z, kind, lim, alpha), wo * gated(wi * g.w, wi * u.w, kind, lim, alpha));
+        }
+        store4(o + i, r);
+    }
+}
+
 }  // namespace citlali
 
 using namespace citlali;
@@ -165,10 +201,18 @@ extern "C" int citlali_expert_gate(const void* gate_up, int in_dtype, const floa
         return kBadShape;
     }
     const int n = E * ff + tail_ff;
-    const int by = (n + 255) / 256;
+    const bool vec = ff % 4 == 0 && tail_ff % 4 == 0 && (E == 0 || run % 4 == 0) && (tail_ff == 0 || tail_run % 4 == 0) &&
+                     (((uintptr_t)gate_up | (uintptr_t)act | (uintptr_t)bias) & 15u) == 0;
+    const int by = vec ? (n / 4 + 255) / 256 : (n + 255) / 256;
     dim3 grid(rows, by < 64 ? by : 64);
     return CITLALI_DISPATCH_FLOAT(in_dtype, TZ, [&] {
         return CITLALI_DISPATCH_FLOAT(act_dtype, TO, [&] {
+            if (vec) {
+                launch_kernel(expert_gate_vec_kernel<TZ, TO>, grid, 256, 0, stream, (const TZ*)gate_up, weights, (TO*)act, E, E > 0 ? ff : 1,
+                              run > 0 ? run : 1, kind, limit, alpha, tail_ff, tail_run > 0 ? tail_run : 1, tail_limit, bias, weight_input,
+                              tail_weights);
+                return CITLALI_LAUNCH_CHECK();
+            }
             launch_kernel(expert_gate_kernel<TZ, TO>, grid, 256, 0, stream, (const TZ*)gate_up, weights, (TO*)act, E, ff,
                           run > 0 ? run : 1, kind, limit, alpha, tail_ff, tail_run > 0 ? tail_run : 1, tail_limit, bias, weight_input,
                           tail_weights);

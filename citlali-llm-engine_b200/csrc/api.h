@@ -103,6 +103,16 @@ int citlali_attention_decode(const void* q, int q_stride, const void* k_pool, co
                              int32_t* counters, size_t counter_ints,
                              int rows, int nq, int nkv, int head_dim, int page_size, int window,
                              int max_positions, float scale, cudaStream_t stream);
+
+// The same on the tensor cores with a value size of its own, a soft cap on the scaled scores, a gate [rows, nq value_dim]
+// (rows gate_stride floats apart), sinks and turned-back outputs, as citlali_attention_prefill takes them.
+int citlali_attention_decode_with_supports(int head_dim, int value_dim, int page_size);
+int citlali_attention_decode_with(const void* q, int q_stride, const void* k_pool, const void* v_pool, const int32_t* page_table,
+                                  int page_table_stride, const int32_t* row_slot, const int32_t* row_pos, void* out,
+                                  int out_stride, float* partial, size_t partial_floats, int32_t* counters, size_t counter_ints,
+                                  int rows, int nq, int nkv, int head_dim, int value_dim, int page_size, int window, float scale,
+                                  float softcap, const float* gate, size_t gate_stride, const float* sink, const float* turns,
+                                  int turn_pairs, cudaStream_t stream);
 void citlali_attention_decode_set_split(int split);
 void citlali_attention_decode_set_by_length(int on, int run_scale_q8);
 void citlali_attention_decode_set_per_warp(int on);
@@ -133,6 +143,13 @@ int citlali_attention_prefill_tc(const void* q, int q_stride, int total_rows,
                                  void* out, int out_stride, int sequences, int max_new,
                                  int nq, int nkv, int head_dim, int page_size, int window, float scale,
                                  int32_t* error_flag, cudaStream_t stream);
+// The same with the options of citlali_attention_prefill (turns 16-byte aligned).
+int citlali_attention_prefill_tc_with(const void* q, int q_stride, int total_rows, const void* k_pool, const void* v_pool,
+                                      int pool_pages, const int32_t* page_table, int page_table_stride, const int32_t* seq_start,
+                                      const int32_t* seq_slot, const int32_t* seq_past, void* out, int out_stride, int sequences,
+                                      int max_new, int nq, int nkv, int head_dim, int page_size, int window, float scale,
+                                      int32_t* error_flag, float softcap, const float* gate, size_t gate_stride, const float* sink,
+                                      const float* turns, int turn_pairs, cudaStream_t stream);
 
 // tokens[r] = argmax of logits[r, :] over finite values, lowest index on ties.
 int citlali_argmax_rows(const float* logits, int32_t* tokens, int rows, int vocab, cudaStream_t stream);

@@ -222,10 +222,50 @@ __device__ __forceinline__ void st_cluster_f32(uint32_t addr, uint32_t rank, flo
 // units), and the blocks of a cluster send their runs of a head to the block that merges that head.
 constexpr int kMaxClusterBlocks = 16;     // blocks per (sequence, head group): a cluster, at most the non-portable size
 
+// What other designs' attention does beside the plain softmax.  cap_out > 0: a score s becomes c tanh(s scale / c), kept in
+// units of log2 (cap_in = 2 log2(e) scale / c, cap_out = c log2(e), and the kernel's scale is 1).  sink: a number a head whose
+// exponential the denominator counts (neither scaled nor capped).  turns [rows, dv / 2] (cos, sin): the output's pairs (m, m +
+// dv / 2), or neighbours, are turned back by the row's angles.  gate: the output's elements times the sigmoids of a row's
+// numbers.  dk, dv: sizes of a key and a value where they are not both the kernel's D (multiples of 8, at most D).
+struct DecodeOptions {
+    float cap_in = 0.0f, cap_out = 0.0f;
+    const float* sink = nullptr;
+    const float2* turns = nullptr;
+    const float* gate = nullptr;
+    size_t gate_stride = 0;
+    int turn_pairs = 0, dk = 0, dv = 0;
+};
+
+__device__ __forceinline__ float sink_share(const DecodeOptions& opt, int head, float M) {      // M in units of log2
+    return opt.sink ? exp2f(opt.sink[head] * 1.4426950408889634f - M) : 0.0f;
+}
+
+// The head's `dv` results value(i): turned back, gated, rounded, stored.
+template <typename Value>
+__device__ __forceinline__ void store_head(const DecodeOptions& opt, int row, int head, int dv, __nv_bfloat16* out_head, int tid, Value value) {
+    auto store = [&](int i, float r) {
+        if (opt.gate) r *= 1.0f / (1.0f + expf(-opt.gate[(size_t)row * opt.gate_stride + (size_t)head * dv + i]));
+        out_head[i] = __float2bfloat16_rn(r);
+    };
+    if (opt.turns) {
+        const int half = dv / 2;
+        for (int m = tid; m < half; m += 128) {
+            const int i = opt.turn_pairs ? 2 * m : m, k = opt.turn_pairs ? i + 1 : i + half;
+            const float2 cs = opt.turns[(size_t)row * half + m];
+            const float u = value(i), v = value(k);
+            store(i, u * cs.x + v * cs.y);
+            store(k, v * cs.x - u * cs.y);
+        }
+    } else {
+        for (int i = tid; i < dv; i += 128) store(i, value(i));
+    }
+}
+
 // One head's (m, l, O) of `runs` consecutive runs of its keys ([run][D + 2] at `base`, m in log2 units), merged in run
 // order into the head's output.  kFromL2: the runs were written by other blocks to global memory (read past L1).
 template <int kBlocks, int D, bool kFromL2>
-__device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfloat16* out_head, int tid) {
+__device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfloat16* out_head, int tid, const DecodeOptions& opt,
+                                           int row, int head, int dv) {
     auto at = [&](size_t i) { return kFromL2 ? __ldcg(base + i) : base[i]; };
     float mz[kBlocks], wz[kBlocks];
 #pragma unroll
@@ -236,7 +276,7 @@ __device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfl
     float M = -INFINITY;
 #pragma unroll
     for (int z = 0; z < kBlocks; ++z) M = fmaxf(M, mz[z]);
-    float L = 0.0f;
+    float L = sink_share(opt, head, M);
 #pragma unroll
     for (int z = 0; z < kBlocks; ++z) {
         const float f = mz[z] == -INFINITY ? 0.0f : exp2f(mz[z] - M);
@@ -244,21 +284,23 @@ __device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfl
         wz[z] = f;
     }
     const float inv = 1.0f / L;
-    for (int i = tid; i < D; i += 128) {
+    store_head(opt, row, head, dv, out_head, tid, [&](int i) {
         float a = 0.0f;
 #pragma unroll
         for (int z = 0; z < kBlocks; ++z)
             if (z < runs && mz[z] != -INFINITY) a = fmaf(at((size_t)z * (D + 2) + 2 + i), wz[z], a);
-        out_head[i] = __float2bfloat16_rn(a * inv);
-    }
+        return a * inv;
+    });
 }
 
 // Block `rank` of a cluster merges heads rank, rank + split, ... over the (m, l, O) of all blocks' runs, which
 // they have sent to `gathered` ([head / split][sender][D + 2]), in rank order.
 template <int kBlocks, int D>
-__device__ __forceinline__ void merge_gathered_heads(const float* gathered, __nv_bfloat16* out_row, int rank, int split, int heads_here, int tid) {
+__device__ __forceinline__ void merge_gathered_heads(const float* gathered, __nv_bfloat16* out_row, int rank, int split, int heads_here, int tid,
+                                                     const DecodeOptions& opt, int row, int head0, int dv) {
     for (int h = rank; h < heads_here; h += split)
-        merge_runs<kBlocks, D, false>(gathered + (size_t)((h / split) * split) * (D + 2), split, out_row + (size_t)h * D, tid);
+        merge_runs<kBlocks, D, false>(gathered + (size_t)((h / split) * split) * (D + 2), split, out_row + (size_t)h * dv, tid, opt, row,
+                                      head0 + h, dv);
 }
 
 constexpr int kMaxRunsByLength = 8;      // blocks a row's keys are dealt to at most when the rows' lengths decide
@@ -277,15 +319,20 @@ constexpr int kMinRunTiles = 16;         // no run shorter than this many pages 
 // kPerWarp (one or few rows: a block an SM at most, clusters of up to sixteen): a warp does not take its 16 keys of
 // every tile the block walks, with the block's two barriers a tile, but a run of 16-key units of its own, fetched into
 // a ring of its own (kStagesKV units) and waited for by the warp alone.  Nothing in the loop holds a warp up for another.
-template <int D, int kStagesKV, bool kByLength, bool kPerWarp = false>
+//
+// kExact: keys and values are D elements; otherwise opt.dk and opt.dv of them, and the tiles' other columns are zeros.
+template <int D, int kStagesKV, bool kByLength, bool kPerWarp = false, bool kExact = true>
 __global__ void __launch_bounds__(128)
 attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                            const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                            const int32_t* __restrict__ page_table, int page_table_stride,
                            const int32_t* __restrict__ row_slot, const int32_t* __restrict__ row_pos,
                            __nv_bfloat16* __restrict__ out, int out_stride, int nq, int nkv, int window,
-                           float scale_log2, float* __restrict__ partial, int* __restrict__ counters, int run_scale_q8) {
+                           float scale_log2, float* __restrict__ partial, int* __restrict__ counters, int run_scale_q8,
+                           const __grid_constant__ DecodeOptions opt) {
     using namespace fa;
+    static_assert(kExact || !kPerWarp, "the form whose warps walk runs of their own takes one size");
+    const int dk = kExact ? D : opt.dk, dv = kExact ? D : opt.dv;
     constexpr int kPage = 64;
     constexpr int kRowBytes = D * 2 + 16;
     constexpr int kTileBytes = kPage * kRowBytes;
@@ -341,14 +388,21 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
 
     auto load_tile = [&](int tile, int buf) {
-        const size_t base = ((size_t)pages[tile] * nkv + g) * kPage * D;
+        const size_t base = ((size_t)pages[tile] * nkv + g) * kPage;
         for (int c = tid; c < kPage * kChunksPerRow; c += 128) {
             const int r = c / kChunksPerRow, ch = c % kChunksPerRow;
-            const size_t src = base + (size_t)r * D + ch * 8;
-            cp_async16(s_k + buf * kTileBytes + r * kRowBytes + ch * 16, k_pool + src);
-            cp_async16(s_v + buf * kTileBytes + r * kRowBytes + ch * 16, v_pool + src);
+            const uint32_t dst = buf * kTileBytes + r * kRowBytes + ch * 16;
+            if (kExact || ch * 8 < dk) cp_async16(s_k + dst, k_pool + (base + r) * dk + ch * 8);
+            if (kExact || ch * 8 < dv) cp_async16(s_v + dst, v_pool + (base + r) * dv + ch * 8);
         }
     };
+    if constexpr (!kExact) {                             // columns no key or value has: zeros, written once
+        for (int c = tid; c < 2 * kStagesKV * kPage * kChunksPerRow; c += 128) {
+            const int r = c / kChunksPerRow, ch = c % kChunksPerRow;          // rows of the key tiles, then of the value tiles
+            if (ch * 8 >= (r < kStagesKV * kPage ? dk : dv))
+                *reinterpret_cast<uint4*>(smem + 16 * kRowBytes + r * kRowBytes + ch * 16) = make_uint4(0, 0, 0, 0);
+        }
+    }
     // Positions and page tables come from the host before the step, and every page but the row's last
     // holds keys and values of earlier steps only.  Unless the row's last page is among this block's
     // first tiles, they are fetched while the kernel ahead of this one (which writes the new token's
@@ -402,7 +456,8 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     for (int c = tid; c < 16 * kChunksPerRow; c += 128) {
         const int r = c / kChunksPerRow, ch = c % kChunksPerRow;
         uint4 w = make_uint4(0, 0, 0, 0);
-        if (r < heads_here) w = *reinterpret_cast<const uint4*>(q + (size_t)row * q_stride + (size_t)(head0 + r) * D + ch * 8);
+        if (r < heads_here && (kExact || ch * 8 < dk))
+            w = *reinterpret_cast<const uint4*>(q + (size_t)row * q_stride + (size_t)(head0 + r) * dk + ch * 8);
         *reinterpret_cast<uint4*>(smem + r * kRowBytes + ch * 16) = w;
     }
     if (!kPerWarp && !early) first_tiles();
@@ -449,6 +504,12 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             ldmatrix_x4(kb + r * kRowBytes + ks * 32 + cbyte, b0, b1, b2, b3);
             mma_16816(s[0], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b0, b1);
             mma_16816(s[1], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b2, b3);
+        }
+        if (opt.cap_out > 0.0f) {                        // tanh z = 1 - 2 / (exp(2 z) + 1)
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s[i][c] = opt.cap_out * (1.0f - __fdividef(2.0f, exp2f(s[i][c] * opt.cap_in) + 1.0f));
         }
         const int key_base = (kPerWarp ? (unit_lo + step) * 16 : tile * kPage + warp * 16) + (lane & 3) * 2;
 #pragma unroll
@@ -537,13 +598,14 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     };
     const int elems = heads_here * (D + 2);
     float* gathered = park + 4 * 16 * (D + 2);       // behind the parked rows: what this block merges
-    __nv_bfloat16* out_row = out + (size_t)row * out_stride + (size_t)head0 * D;
+    __nv_bfloat16* out_row = out + (size_t)row * out_stride + (size_t)head0 * dv;
     if (split == 1) {
         for (int e = tid; e < elems; e += 128) gathered[e] = folded(e);
         __syncthreads();
-        for (int e = tid; e < heads_here * D; e += 128) {
-            const int h = e / D, i = e % D;
-            out_row[(size_t)h * D + i] = __float2bfloat16_rn(gathered[h * (D + 2) + 2 + i] * (1.0f / gathered[h * (D + 2) + 1]));
+        for (int h = 0; h < heads_here; ++h) {
+            const float* mine = gathered + h * (D + 2);
+            const float inv = 1.0f / (mine[1] + sink_share(opt, head0 + h, mine[0]));
+            store_head(opt, row, head0 + h, dv, out_row + (size_t)h * dv, tid, [&](int i) { return mine[2 + i] * inv; });
         }
         return;
     }
@@ -568,7 +630,7 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         __threadfence();
         for (int h = 0; h < heads_here; ++h)
             merge_runs<kMaxRunsByLength, D, true>(partial + ((size_t)row * nq + head0 + h) * chunks * (D + 2), split,
-                                                  out_row + (size_t)h * D, tid);
+                                                  out_row + (size_t)h * dv, tid, opt, row, head0 + h, dv);
         return;
     }
     // Head h is merged by block h % split.  Every block sends its (m, l, O) of a head into that block's shared
@@ -584,10 +646,10 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     }
     cluster_arrive();
     cluster_wait();
-    if (split <= 2) merge_gathered_heads<2, D>(gathered, out_row, rank, split, heads_here, tid);
-    else if (split <= 4) merge_gathered_heads<4, D>(gathered, out_row, rank, split, heads_here, tid);
-    else if (split <= 8) merge_gathered_heads<8, D>(gathered, out_row, rank, split, heads_here, tid);
-    else merge_gathered_heads<kMaxClusterBlocks, D>(gathered, out_row, rank, split, heads_here, tid);
+    if (split <= 2) merge_gathered_heads<2, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else if (split <= 4) merge_gathered_heads<4, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else if (split <= 8) merge_gathered_heads<8, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else merge_gathered_heads<kMaxClusterBlocks, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
 }
 
 static int g_forced_split = 0;     // > 0: blocks per (sequence, head group), for tuning
@@ -596,16 +658,16 @@ static int g_per_warp = 1;         // 0: never the kernel whose warps walk runs 
 static int g_run_scale_q8 = 160;   // by-length kernel: a run's length in 1/256 of the mean length of the step's rows
 static int g_by_length = 1;        // 0: never deal a row's pages out by length
 
-template <int D, int kStagesKV, bool kByLength = false, bool kPerWarp = false>
+template <int D, int kStagesKV, bool kByLength = false, bool kPerWarp = false, bool kExact = true>
 static int launch_tc_stages(const void* q, int q_stride, const void* k_pool, const void* v_pool, const int32_t* page_table,
                      int page_table_stride, const int32_t* row_slot, const int32_t* row_pos, void* out, int out_stride,
-                     int rows, int nq, int nkv, int window, float scale, int split, cudaStream_t stream,
+                     int rows, int nq, int nkv, int window, float scale, int split, const DecodeOptions& opt, cudaStream_t stream,
                      float* partial = nullptr, int* counters = nullptr) {
     constexpr int tiles = (16 + 2 * kStagesKV * 64) * (D * 2 + 16);
     // the query rows, the four warps' parked rows, and behind them what the cluster's blocks send (at most 31 runs)
     constexpr int park = 16 * (D * 2 + 16) + (4 * 16 + 32) * (D + 2) * 4;
     constexpr int smem = tiles > park ? tiles : park;
-    auto kernel = attention_decode_tc_kernel<D, kStagesKV, kByLength, kPerWarp>;
+    auto kernel = attention_decode_tc_kernel<D, kStagesKV, kByLength, kPerWarp, kExact>;
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -622,7 +684,7 @@ static int launch_tc_stages(const void* q, int q_stride, const void* k_pool, con
     launch_kernel_clustered(kernel, grid, 128, smem, kByLength ? 1 : split, stream, (const __nv_bfloat16*)q, q_stride,
                             (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_table, page_table_stride,
                             row_slot, row_pos, (__nv_bfloat16*)out, out_stride, nq, nkv, window,
-                            scale * 1.4426950408889634f, partial, counters, g_run_scale_q8);
+                            opt.cap_out > 0.0f ? 1.0f : scale * 1.4426950408889634f, partial, counters, g_run_scale_q8, opt);
     return CITLALI_LAUNCH_CHECK();
 }
 
@@ -630,10 +692,10 @@ static int launch_tc_stages(const void* q, int q_stride, const void* k_pool, con
 // head size 128, 8 key/value heads, 4,096 cached tokens: one sequence 8 blocks, eight sequences 4, sixty-four
 // sequences 1 (no merging at all once the grid fills the GPU twice over).  The choice depends on the batch
 // alone, never on the sequences' lengths, so a captured launch stays valid.
-template <int D>
+template <int D, bool kExact = true>
 static int launch_tc(const void* q, int q_stride, const void* k_pool, const void* v_pool, const int32_t* page_table,
                      int page_table_stride, const int32_t* row_slot, const int32_t* row_pos, void* out, int out_stride,
-                     int rows, int nq, int nkv, int window, float scale, cudaStream_t stream,
+                     int rows, int nq, int nkv, int window, float scale, const DecodeOptions& opt, cudaStream_t stream,
                      float* partial, size_t partial_floats, int* counters, size_t counter_ints) {
     const int group = nq / nkv;
     const long pairs = (long)rows * nkv * ((group + 15) / 16);
@@ -653,25 +715,25 @@ static int launch_tc(const void* q, int q_stride, const void* k_pool, const void
         if (runs > kMaxRunsByLength) runs = kMaxRunsByLength;
         while (runs > 1 && (size_t)rows * nq * runs * (D + 2) > partial_floats) --runs;
         if (runs > 1)
-            return launch_tc_stages<D, kKvStages, true>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot,
-                                                        row_pos, out, out_stride, rows, nq, nkv, window, scale, runs, stream,
-                                                        partial, counters);
+            return launch_tc_stages<D, kKvStages, true, false, kExact>(q, q_stride, k_pool, v_pool, page_table, page_table_stride,
+                                                                       row_slot, row_pos, out, out_stride, rows, nq, nkv, window, scale,
+                                                                       runs, opt, stream, partial, counters);
     }
     // One or two rows (at most a block an SM): every warp walks a run of 16-key units of its own, three units in flight
     // a warp.  Measured against the block-wide walk at batch 1: 8.1 against 8.5 us at 4,000 cached tokens, 11.5 against
     // 13.5 at 8,000, 18.0 against 23.4 at 16,000 (batch 2: 10.8 / 12.5, 17.3 / 21.6, 30.3 / 39.7); with more rows, where
     // the launch is bound by bandwidth, it gains nothing (batch 8 at 4,000: 23.9 either way).  A ring of six units a
     // warp (one block an SM) lost 3.5 us at every length: the next launch's blocks no longer fit beside this one's.
-    if constexpr (D <= 128) {
+    if constexpr (D <= 128 && kExact) {
         if (g_per_warp && pairs * split <= device_sm_count())
             return launch_tc_stages<D, kKvStages, false, true>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, out,
-                                                       out_stride, rows, nq, nkv, window, scale, split, stream);
+                                                       out_stride, rows, nq, nkv, window, scale, split, opt, stream);
         if (pairs * split <= 80)          // more blocks than that, each filling an SM, no longer fit cluster by cluster
             return launch_tc_stages<D, 6>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, out,
-                                          out_stride, rows, nq, nkv, window, scale, split, stream);
+                                          out_stride, rows, nq, nkv, window, scale, split, opt, stream);
     }
-    return launch_tc_stages<D, kKvStages>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, out,
-                                          out_stride, rows, nq, nkv, window, scale, split, stream);
+    return launch_tc_stages<D, kKvStages, false, false, kExact>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, out,
+                                          out_stride, rows, nq, nkv, window, scale, split, opt, stream);
 }
 
 template <int EPL, int GT>
@@ -766,7 +828,7 @@ extern "C" int citlali_attention_decode(const void* q, int q_stride, const void*
         // pages of 64 and a head size the tensor-core kernel has: in steps of few rows its blocks merge their
         // partial results through distributed shared memory and the scratch is not used
 #define CITLALI_TC(DD) case DD: return launch_tc<DD>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, \
-                                                      out, out_stride, rows, nq, nkv, window, scale, stream, partial, \
+                                                      out, out_stride, rows, nq, nkv, window, scale, DecodeOptions(), stream, partial, \
                                                       partial_floats, counters, counter_ints)
         switch (head_dim) {
             CITLALI_TC(16); CITLALI_TC(32); CITLALI_TC(48); CITLALI_TC(64); CITLALI_TC(80); CITLALI_TC(96); CITLALI_TC(112);
@@ -811,4 +873,67 @@ extern "C" int citlali_attention_decode(const void* q, int q_stride, const void*
     launch_kernel(attention_decode_combine_kernel, grid, 128, (size_t)(max_chunks + 1) * sizeof(float), stream, partial, max_chunks, row_pos, (__nv_bfloat16*)out, out_stride,
                                                               nq, head_dim, chunk_keys, window);
     return CITLALI_LAUNCH_CHECK();
+}
+
+// 1 if citlali_attention_decode_with has a kernel for keys of d and values of vd elements.
+extern "C" int citlali_attention_decode_with_supports(int d, int vd, int page_size) {
+    return page_size == 64 && d > 0 && vd > 0 && d % 8 == 0 && vd % 8 == 0 && d <= 256 && vd <= 256;
+}
+
+// citlali_attention_decode on the tensor cores with what other designs' attention does beside the plain softmax.
+extern "C" int citlali_attention_decode_with(const void* q, int q_stride, const void* k_pool, const void* v_pool,
+                                             const int32_t* page_table, int page_table_stride, const int32_t* row_slot,
+                                             const int32_t* row_pos, void* out, int out_stride, float* partial,
+                                             size_t partial_floats, int32_t* counters, size_t counter_ints, int rows, int nq,
+                                             int nkv, int head_dim, int value_dim, int page_size, int window, float scale,
+                                             float softcap, const float* gate, size_t gate_stride, const float* sink,
+                                             const float* turns, int turn_pairs, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || rows > 65535 || nq > 65535) {
+        set_last_error("attention_decode_with: %d query heads over %d key/value heads, %d rows", nq, nkv, rows);
+        return kBadShape;
+    }
+    if (!citlali_attention_decode_with_supports(head_dim, value_dim, page_size)) {
+        set_last_error("attention_decode_with: no kernel for keys of %d and values of %d with pages of %d (multiples of 8 up to 256, "
+                       "pages of 64)", head_dim, value_dim, page_size);
+        return kBadShape;
+    }
+    if (q_stride % 8 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)turns & 7u)) {
+        set_last_error("attention_decode_with: query rows must be 16-byte aligned (row pitch %d elements)", q_stride);
+        return kBadAlignment;
+    }
+    DecodeOptions opt;
+    opt.cap_in = softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f;
+    opt.cap_out = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
+    opt.sink = sink;
+    opt.turns = (const float2*)turns;
+    opt.gate = gate;
+    opt.gate_stride = gate_stride;
+    opt.turn_pairs = turn_pairs;
+    opt.dk = head_dim;
+    opt.dv = value_dim;
+#define CITLALI_TC(DD, EX) return launch_tc<DD, EX>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, \
+                                                      out, out_stride, rows, nq, nkv, window, scale, opt, stream, partial, \
+                                                      partial_floats, counters, counter_ints)
+    if (head_dim == value_dim) {
+        switch (head_dim) {
+            case 16: CITLALI_TC(16, true);
+            case 32: CITLALI_TC(32, true);
+            case 48: CITLALI_TC(48, true);
+            case 64: CITLALI_TC(64, true);
+            case 80: CITLALI_TC(80, true);
+            case 96: CITLALI_TC(96, true);
+            case 112: CITLALI_TC(112, true);
+            case 128: CITLALI_TC(128, true);
+            case 256: CITLALI_TC(256, true);
+            default: break;
+        }
+    }
+    const int widest = head_dim > value_dim ? head_dim : value_dim;
+    if (widest <= 32) CITLALI_TC(32, false);
+    if (widest <= 64) CITLALI_TC(64, false);
+    if (widest <= 96) CITLALI_TC(96, false);
+    if (widest <= 128) CITLALI_TC(128, false);
+    CITLALI_TC(256, false);
+#undef CITLALI_TC
 }

@@ -39,6 +39,13 @@
 // src/compute/cuda/kernels.cu:545-649): s = q.k / sqrt(d), keys lo..p for the token at position
 // p, query head j reads key/value head j / (heads / kv_heads); softmax and sums in float.
 // Every mbarrier wait is bounded and reports through the error word.
+//
+// A second instance of the kernel (kWith) does what other designs' attention has beside the plain softmax: a soft cap on the
+// scaled scores (each score, as it comes out of tensor memory, becomes c tanh(s scale / c) in units of log2, ahead of the
+// mask), a sink a head (added to the row's sum at the end), an output turned back by the row's own angles (the other half of
+// a pair of halves lies in the same lane of tensor memory) and a gate on the output.  Scores under a cap of up to 69 lie
+// within 2^100 of one: exponentials are then taken against zero, no maximum is looked for, and the two warps of a row's halves
+// do not meet before the end.
 #include "api.h"
 #include "common.cuh"
 #include "tc_common.cuh"
@@ -217,6 +224,13 @@ struct Params {
     int pair_heads;                      // 1: the two query tiles are heads 2x, 2x+1; 0: row tiles 2y, 2y+1 of head x
     float scale_log2;
     int32_t* error_flag;
+    // kWith only: cap_in = 2 log2(e) scale / cap and cap_out = cap log2(e) (scale_log2 is then 1; 0: no cap); sink [nq]; turns
+    // [rows, 64] (cos, sin) of the pairs (m, m + 64), or with turn_pairs (2m, 2m + 1); gate, rows gate_stride floats apart
+    float cap_in, cap_out;
+    int fixed_reference;                 // capped scores lie in +-cap_out, small enough that zero serves as every row's reference
+    const float* sink; const float2* turns; const float* gate;
+    size_t gate_stride;
+    int turn_pairs;
 };
 
 // One of the block's two query tiles: its head, its first row within the sequence's new tokens, and the
@@ -226,6 +240,13 @@ struct QueryTile {
     __device__ bool reads(int t) const { return t >= tile_lo && t <= tile_hi; }
 };
 
+__device__ __forceinline__ float fast_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <bool kWith>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, Params p) {
@@ -432,7 +453,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int warp_pos = past + me.q0 + quarter * 32;
         const uint32_t meet = smem_u32(&pair_bar[b][quarter]);
         uint32_t meetings = 0;
-        float m_ref = -INFINITY, l = 0.0f;                    // the row's reference maximum (raw score units), this half's sum
+        const bool fixed = kWith && p.fixed_reference != 0;
+        float m_ref = fixed ? 0.0f : -INFINITY, l = 0.0f;     // the row's reference maximum (raw score units), this half's sum
         bool ok = true;
         // Both warps of the pair arrive and wait; what either wrote to shared memory before is visible to both after.
         auto meet_partner = [&]() -> bool {
@@ -450,6 +472,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             uint32_t pk[32];                                  // P of this half row, two bfloat16 a register
             uint32_t a[16], bb[16];
             auto mask16 = [&](uint32_t (&h)[16], int c_base) {
+                if constexpr (kWith) {
+                    if (p.cap_out > 0.0f) {                   // tanh z = 1 - 2 / (exp(2 z) + 1)
+#pragma unroll
+                        for (int c = 0; c < 16; ++c)
+                            h[c] = __float_as_uint(fmaf(-2.0f * p.cap_out, fast_rcp(ex2(__uint_as_float(h[c]) * p.cap_in) + 1.0f), p.cap_out));
+                    }
+                }
                 if (masked) {
 #pragma unroll
                     for (int c = 0; c < 16; ++c) {
@@ -458,7 +487,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     }
                 }
             };
-            bool two_pass = t == 0;
+            bool two_pass = t == 0 && !fixed;
             if (!two_pass) {
                 // One pass, 16 scores at a time while the next 16 are on their way from tensor memory.  A P above
                 // 2^15 makes the sum exceed 2^15, and a sum above 2^15 needs a P above 2^8: past that the
@@ -493,12 +522,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tmem_ld_wait16(bb);
                 chunk(bb, 48);
                 const float tile_sum = (s0 + s1) + (s2 + s3);
+                if (fixed) {
+                    l += tile_sum;
+                } else {
                 const bool in_range = tile_sum <= 32768.0f && m_ref != -INFINITY;      // false for inf and NaN too
                 const bool mine = __any_sync(0xffffffffu, !in_range);
                 if (lane == 0) pair_vote[b][quarter][half] = mine ? 1 : 0;
                 if (!meet_partner()) { ok = false; break; }
                 two_pass = mine || pair_vote[b][quarter][half ^ 1] != 0;
                 if (!two_pass) l += tile_sum;
+                }
             }
             if (two_pass) {
                 // The row's maximum first (this half's, then the other's through shared memory), then the exponentials
@@ -581,14 +614,59 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         if (ok && tiles > 0 && mbar_wait(smem_u32(&o_done[b]), 0, abort_flag, p.error_flag, 209)) {
             tc_fence_after();
+            if constexpr (kWith) {
+                if (p.sink && m_ref != -INFINITY) l += ex2(p.sink[me.head] * 1.4426950408889634f - m_ref * p.scale_log2);
+            }
             const float inv = l > 0.0f ? 1.0f / l : 0.0f;
             const bool store = me.q0 + r < n_new;
             __nv_bfloat16* dst = p.out + (size_t)(row0 + me.q0 + r) * p.out_stride + (size_t)me.head * kD + half * kHalfKeys;
 #pragma unroll 1
             for (int c0 = 0; c0 < kHalfKeys; c0 += 16) {
                 uint32_t ov[16];
+                [[maybe_unused]] uint32_t a[16];
                 tmem_ld16(sub + kColO + half * kHalfKeys + c0, ov);
                 tmem_ld_wait16(ov);
+                if constexpr (kWith) {
+                    if (p.turns && !p.turn_pairs) {           // the pair's other element: the same place in the other half
+                        tmem_ld16(sub + kColO + (half ^ 1) * kHalfKeys + c0, a);
+                        tmem_ld_wait16(a);
+                    }
+                    if (store) {
+                        const size_t row = row0 + me.q0 + r;
+                        if (p.turns) {
+                            const float2* t = p.turns + row * kHalfKeys;
+                            if (!p.turn_pairs) {
+                                const float sign = half ? -1.0f : 1.0f;                 // u c + v s, v c - u s
+#pragma unroll
+                                for (int c = 0; c < 16; c += 2) {
+                                    const float4 cs = *reinterpret_cast<const float4*>(t + c0 + c);
+                                    ov[c] = __float_as_uint(fmaf(__uint_as_float(a[c]), sign * cs.y, __uint_as_float(ov[c]) * cs.x));
+                                    ov[c + 1] = __float_as_uint(fmaf(__uint_as_float(a[c + 1]), sign * cs.w, __uint_as_float(ov[c + 1]) * cs.z));
+                                }
+                            } else {
+#pragma unroll
+                                for (int c = 0; c < 16; c += 2) {
+                                    const float2 cs = t[(half * kHalfKeys + c0 + c) >> 1];
+                                    const float u = __uint_as_float(ov[c]), v = __uint_as_float(ov[c + 1]);
+                                    ov[c] = __float_as_uint(fmaf(v, cs.y, u * cs.x));
+                                    ov[c + 1] = __float_as_uint(fmaf(-u, cs.y, v * cs.x));
+                                }
+                            }
+                        }
+                        if (p.gate) {
+                            const float* gt = p.gate + row * p.gate_stride + (size_t)me.head * kD + half * kHalfKeys + c0;
+#pragma unroll
+                            for (int c = 0; c < 16; c += 4) {
+                                const float4 z = *reinterpret_cast<const float4*>(gt + c);
+                                const float k = -1.4426950408889634f;
+                                ov[c] = __float_as_uint(__fdividef(__uint_as_float(ov[c]), 1.0f + ex2(k * z.x)));
+                                ov[c + 1] = __float_as_uint(__fdividef(__uint_as_float(ov[c + 1]), 1.0f + ex2(k * z.y)));
+                                ov[c + 2] = __float_as_uint(__fdividef(__uint_as_float(ov[c + 2]), 1.0f + ex2(k * z.z)));
+                                ov[c + 3] = __float_as_uint(__fdividef(__uint_as_float(ov[c + 3]), 1.0f + ex2(k * z.w)));
+                            }
+                        }
+                    }
+                }
                 if (store) {
 #pragma unroll
                     for (int c = 0; c < 16; c += 8) {
@@ -628,15 +706,12 @@ extern "C" int citlali_attention_prefill_tc_supports(int head_dim, int page_size
     return head_dim == fatc::kD && page_size == fatc::kPage;
 }
 
-// As citlali_attention_prefill, on tcgen05, for head size 128 and pages of 64.  `total_rows` is the
-// number of rows of q (all sequences), `pool_pages` the number of pages of the layer's pools.
-extern "C" int citlali_attention_prefill_tc(const void* q, int q_stride, int total_rows,
-                                            const void* k_pool, const void* v_pool, int pool_pages,
-                                            const int32_t* page_table, int page_table_stride,
-                                            const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
-                                            void* out, int out_stride, int sequences, int max_new,
-                                            int nq, int nkv, int head_dim, int page_size, int window, float scale,
-                                            int32_t* error_flag, cudaStream_t stream) {
+static int launch_prefill_tc(const void* q, int q_stride, int total_rows, const void* k_pool, const void* v_pool, int pool_pages,
+                             const int32_t* page_table, int page_table_stride, const int32_t* seq_start, const int32_t* seq_slot,
+                             const int32_t* seq_past, void* out, int out_stride, int sequences, int max_new, int nq, int nkv,
+                             int head_dim, int page_size, int window, float scale, int32_t* error_flag, bool with, float softcap,
+                             const float* gate, size_t gate_stride, const float* sink, const float* turns, int turn_pairs,
+                             cudaStream_t stream) {
     if (sequences <= 0 || max_new <= 0) return 0;
     if (!citlali_attention_prefill_tc_supports(head_dim, page_size)) {
         set_last_error("attention_prefill_tc: head size %d with pages of %d is not taken (128 and 64 only)", head_dim, page_size);
@@ -647,7 +722,7 @@ extern "C" int citlali_attention_prefill_tc(const void* q, int q_stride, int tot
         return kBadShape;
     }
     if (q_stride % 8 != 0 || out_stride % 8 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 15u) ||
-        ((uintptr_t)k_pool & 15u) || ((uintptr_t)v_pool & 15u)) {
+        ((uintptr_t)k_pool & 15u) || ((uintptr_t)v_pool & 15u) || ((uintptr_t)turns & 15u) || ((uintptr_t)gate & 15u) || (gate && gate_stride % 4 != 0)) {
         set_last_error("attention_prefill_tc: rows of q and out must be 16-byte aligned");
         return kBadAlignment;
     }
@@ -664,17 +739,49 @@ extern "C" int citlali_attention_prefill_tc(const void* q, int q_stride, int tot
     p.nq = nq; p.nkv = nkv; p.window = window;
     // two heads of a key/value group share a block when groups have an even number of heads, else two row tiles
     p.pair_heads = (nq / nkv) % 2 == 0 ? 1 : 0;
-    p.scale_log2 = scale * 1.4426950408889634f;
+    const float log2e = 1.4426950408889634f;
+    p.scale_log2 = softcap > 0.0f ? 1.0f : scale * log2e;
     p.error_flag = error_flag;
+    p.cap_in = softcap > 0.0f ? 2.0f * log2e * scale / softcap : 0.0f;
+    p.cap_out = softcap > 0.0f ? softcap * log2e : 0.0f;
+    p.fixed_reference = p.cap_out > 0.0f && p.cap_out <= 100.0f ? 1 : 0;
+    p.sink = sink; p.turns = (const float2*)turns; p.gate = gate; p.gate_stride = gate_stride; p.turn_pairs = turn_pairs;
     const size_t smem = (size_t)6 * fatc::kTileBytes + 1024;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(fatc::attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    auto kernel = with ? fatc::attention_prefill_tc_kernel<true> : fatc::attention_prefill_tc_kernel<false>;
+    static bool configured[2] = {false, false};
+    if (!configured[with]) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        configured = true;
+        configured[with] = true;
     }
     const int row_tiles = (max_new + fatc::kTileQ - 1) / fatc::kTileQ;
     dim3 grid(p.pair_heads ? nq / 2 : nq, p.pair_heads ? row_tiles : (row_tiles + 1) / 2, sequences);
-    launch_kernel(fatc::attention_prefill_tc_kernel, grid, fatc::kThreads, smem, stream, mq, mk, mv, p);
+    launch_kernel(kernel, grid, fatc::kThreads, smem, stream, mq, mk, mv, p);
     return CITLALI_LAUNCH_CHECK();
+}
+
+// As citlali_attention_prefill, on tcgen05, for head size 128 and pages of 64.  `total_rows` is the
+// number of rows of q (all sequences), `pool_pages` the number of pages of the layer's pools.
+extern "C" int citlali_attention_prefill_tc(const void* q, int q_stride, int total_rows,
+                                            const void* k_pool, const void* v_pool, int pool_pages,
+                                            const int32_t* page_table, int page_table_stride,
+                                            const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
+                                            void* out, int out_stride, int sequences, int max_new,
+                                            int nq, int nkv, int head_dim, int page_size, int window, float scale,
+                                            int32_t* error_flag, cudaStream_t stream) {
+    return launch_prefill_tc(q, q_stride, total_rows, k_pool, v_pool, pool_pages, page_table, page_table_stride, seq_start, seq_slot,
+                             seq_past, out, out_stride, sequences, max_new, nq, nkv, head_dim, page_size, window, scale, error_flag,
+                             false, 0.0f, nullptr, 0, nullptr, nullptr, 0, stream);
+}
+
+extern "C" int citlali_attention_prefill_tc_with(const void* q, int q_stride, int total_rows, const void* k_pool, const void* v_pool,
+                                                 int pool_pages, const int32_t* page_table, int page_table_stride,
+                                                 const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past, void* out,
+                                                 int out_stride, int sequences, int max_new, int nq, int nkv, int head_dim,
+                                                 int page_size, int window, float scale, int32_t* error_flag, float softcap,
+                                                 const float* gate, size_t gate_stride, const float* sink, const float* turns,
+                                                 int turn_pairs, cudaStream_t stream) {
+    return launch_prefill_tc(q, q_stride, total_rows, k_pool, v_pool, pool_pages, page_table, page_table_stride, seq_start, seq_slot,
+                             seq_past, out, out_stride, sequences, max_new, nq, nkv, head_dim, page_size, window, scale, error_flag,
+                             true, softcap, gate, gate_stride, sink, turns, turn_pairs, stream);
 }

@@ -41,11 +41,22 @@ __global__ void embed_rows_kernel(const TW* __restrict__ table, const int32_t* _
     }
 }
 
+__device__ __forceinline__ void load4_as_float(const float* p, float (&v)[4]) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void load4_as_float(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(w.x << 16); v[1] = __uint_as_float(w.x & 0xffff0000u);
+    v[2] = __uint_as_float(w.y << 16); v[3] = __uint_as_float(w.y & 0xffff0000u);
+}
+
 // x = E[token] * scale + P[row] * pair_scale with row = (previous token * mul_prev + token * mul_cur) mod buckets, and row
 // `buckets` for a sequence's first token.  The token before a sequence's first row of the step is what the sequence kept
 // (state[slot], read only past position 0); the block of that row leaves the sequence's last token of the step there.
 template <typename TW>
-__global__ void embed_rows_paired_kernel(const TW* __restrict__ table, const TW* __restrict__ pairs,
+__global__ void __launch_bounds__(1024)
+embed_rows_paired_kernel(const TW* __restrict__ table, const TW* __restrict__ pairs,
                                          const int32_t* __restrict__ tokens, const int32_t* __restrict__ row_slot,
                                          const int32_t* __restrict__ row_pos, const int32_t* __restrict__ seq_start, int sequences,
                                          int32_t* __restrict__ state, float* __restrict__ out, int hidden, int vocab, int buckets,
@@ -79,6 +90,18 @@ __global__ void embed_rows_paired_kernel(const TW* __restrict__ table, const TW*
     const TW* src = table + (size_t)(ok ? tok : 0) * hidden;
     const TW* pair = pairs + (size_t)pair_row * hidden;
     float* dst = out + (size_t)row * hidden;
+    if (hidden % 4 == 0) {                                    // rows start on 8-byte (bfloat16) or 16-byte boundaries
+        for (int i = threadIdx.x * 4; i < hidden; i += blockDim.x * 4) {
+            float a[4], b[4];
+            load4_as_float(src + i, a);
+            load4_as_float(pair + i, b);
+            float4 v = make_float4(fmaf(b[0], pair_scale, a[0] * scale), fmaf(b[1], pair_scale, a[1] * scale),
+                                   fmaf(b[2], pair_scale, a[2] * scale), fmaf(b[3], pair_scale, a[3] * scale));
+            if (!ok) v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            *reinterpret_cast<float4*>(dst + i) = v;
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? fmaf(ldf(pair, i), pair_scale, ldf(src, i) * scale) : 0.0f;
 }
 
@@ -273,8 +296,14 @@ extern "C" int citlali_embed_rows_paired(const void* table, const void* pairs, i
                        mul_prev, mul_cur);
         return kBadShape;
     }
+    if (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out) & 15u) {
+        set_last_error("embed_rows_paired: the tables and the output must start on 16-byte boundaries");
+        return kBadAlignment;
+    }
+    int threads = (hidden / 4 + 31) / 32 * 32;
+    threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
     return CITLALI_DISPATCH_FLOAT(table_dtype, TW, [&] {
-        launch_kernel(embed_rows_paired_kernel<TW>, rows, 256, 0, stream, (const TW*)table, (const TW*)pairs, tokens, row_slot,
+        launch_kernel(embed_rows_paired_kernel<TW>, rows, threads, 0, stream, (const TW*)table, (const TW*)pairs, tokens, row_slot,
                       row_pos, seq_start, sequences, state, out, hidden, vocab, buckets, mul_prev, mul_cur, scale, pair_scale,
                       error_flag);
         return CITLALI_LAUNCH_CHECK();

@@ -18,6 +18,7 @@ namespace citlali {
 
 constexpr int kPiece = 512;            // elements of a part one warp sums
 constexpr int kNormThreads = 256;
+constexpr int kWideThreads = 1024;     // at most, for kernels whose blocks have one row (or a sequence's kept rows) to themselves
 constexpr int kMaxTaps = 16;
 
 
@@ -44,6 +45,9 @@ __device__ __forceinline__ float4 get4(const TG* p) {
     }
 }
 
+// a b c, every product rounded (never part of a fused multiply-add: a row h is the same wherever it is formed)
+__device__ __forceinline__ float rounded3(float a, float b, float c) { return __fmul_rn(__fmul_rn(a, b), c); }
+
 // inv[r * groups + g] = 1 / sqrt(mean of squares of part g of source row r + eps) for `n` rows; `row_of(r)` names the row (below
 // zero: none, inv stays unset).  `sums` holds n * groups * pieces floats.  Ends with a barrier.
 template <bool VEC, typename RowOf>
@@ -51,25 +55,45 @@ __device__ __forceinline__ void inverse_roots(const float* __restrict__ x, int h
                                               float* inv, RowOf row_of) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int part = hidden / groups, pieces = pieces_of(part), per_row = groups * pieces;
-    for (int task = warp; task < n * per_row; task += warps) {
-        const int r = task / per_row, g = (task % per_row) / pieces, p = task % pieces;
-        const int row = row_of(r);
-        if (row < 0) continue;
-        const int i0 = p * kPiece, i1 = min(part, i0 + kPiece);
-        const float* src = x + (size_t)row * hidden + (size_t)g * part;
-        float ss = 0.0f;
-        if constexpr (VEC) {
+    if constexpr (VEC) {
+        constexpr int U = 2, Q = kPiece / 128;                 // pieces in flight a warp, 16-byte words of one a lane holds
+        for (int t0 = warp; t0 < n * per_row; t0 += warps * U) {
+            float4 v[U][Q];
 #pragma unroll
-            for (int k = 0; k < kPiece / 128; ++k) {
-                const int i = i0 + (k * 32 + lane) * 4;
-                const float4 v = i < i1 ? *reinterpret_cast<const float4*>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-                ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+            for (int u = 0; u < U; ++u) {
+                const int task = t0 + u * warps;
+                const int r = task / per_row, g = (task % per_row) / pieces, i0 = task % pieces * kPiece;
+                const int row = task < n * per_row ? row_of(r) : -1;
+                const float* src = x + (size_t)max(row, 0) * hidden + (size_t)g * part;
+#pragma unroll
+                for (int k = 0; k < Q; ++k) {
+                    const int i = i0 + (k * 32 + lane) * 4;
+                    v[u][k] = row >= 0 && i < min(part, i0 + kPiece) ? *reinterpret_cast<const float4*>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
             }
-        } else {
-            for (int i = i0 + lane; i < i1; i += 32) ss = fmaf(src[i], src[i], ss);
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int k = 0; k < Q; ++k) {
+                    ss = fmaf(v[u][k].x, v[u][k].x, ss); ss = fmaf(v[u][k].y, v[u][k].y, ss);
+                    ss = fmaf(v[u][k].z, v[u][k].z, ss); ss = fmaf(v[u][k].w, v[u][k].w, ss);
+                }
+                ss = warp_sum(ss);
+                if (lane == 0 && t0 + u * warps < n * per_row) sums[t0 + u * warps] = ss;
+            }
         }
-        ss = warp_sum(ss);
-        if (lane == 0) sums[task] = ss;
+    } else {
+        for (int task = warp; task < n * per_row; task += warps) {
+            const int r = task / per_row, g = (task % per_row) / pieces, i0 = task % pieces * kPiece;
+            const int row = row_of(r), i1 = min(part, i0 + kPiece);
+            if (row < 0) continue;
+            const float* src = x + (size_t)row * hidden + (size_t)g * part;
+            float ss = 0.0f;
+            for (int i = i0 + lane; i < i1; i += 32) ss = fmaf(src[i], src[i], ss);
+            ss = warp_sum(ss);
+            if (lane == 0) sums[task] = ss;
+        }
     }
     __syncthreads();
     for (int t = threadIdx.x; t < n * groups; t += blockDim.x) {
@@ -105,22 +129,22 @@ group_rms_norm_kernel(const float* __restrict__ x, const TG* __restrict__ gain, 
     }
 }
 
-// A block takes `R` consecutive rows of the step and the taps - 1 rows ahead of them.
-template <typename TG, typename TO, int TAPS>
-__global__ void __launch_bounds__(kNormThreads)
+// A block takes R consecutive rows of the step and the taps - 1 rows ahead of them.
+template <typename TG, typename TO, int TAPS, int R>
+__global__ void __launch_bounds__(R == 1 ? kWideThreads : kNormThreads)
 group_norm_conv_vec_kernel(const float* __restrict__ x, const TG* __restrict__ gain, const float* __restrict__ taps_w,
                            float* __restrict__ state, size_t state_stride, const int32_t* __restrict__ row_slot,
-                           TO* __restrict__ h_out, TO* __restrict__ c_out, int rows, int hidden, int groups, float eps, int R) {
+                           TO* __restrict__ h_out, TO* __restrict__ c_out, int rows, int hidden, int groups, float eps) {
     extern __shared__ float sm[];
     dependents_may_launch();
     wait_for_predecessor();
     constexpr int BACK = TAPS - 1;
     const int part = hidden / groups, per = groups * pieces_of(part);
-    float* inv = sm + (size_t)(R + BACK) * per;                // local row r stands for row r0 - BACK + r
+    float* inv = sm + (size_t)(R + BACK) * per;                // local row r stands for row r0 - before + r
     const int r0 = blockIdx.x * R, nr = min(R, rows - r0);
-    inverse_roots<true>(x, hidden, groups, eps, nr + BACK, sm, inv, [&](int r) { return r0 - BACK + r; });
     int before = 0;                                            // rows ahead of r0 that belong to its sequence
     while (before < BACK && r0 - before - 1 >= 0 && row_slot[r0 - before - 1] == row_slot[r0]) ++before;
+    inverse_roots<true>(x, hidden, groups, eps, before + nr, sm, inv, [&](int r) { return r0 - before + r; });
     for (int c = threadIdx.x * 4; c < hidden; c += blockDim.x * 4) {
         const float4 g = get4(gain + c);
         const int grp = c / part;
@@ -135,29 +159,35 @@ group_norm_conv_vec_kernel(const float* __restrict__ x, const TG* __restrict__ g
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) w[j] = make_float4(t[j], t[TAPS + j], t[2 * TAPS + j], t[3 * TAPS + j]);
         }
-        auto normed = [&](int row) {
-            const float4 v = *reinterpret_cast<const float4*>(x + (size_t)row * hidden + c);
-            const float k = inv[(row - r0 + BACK) * groups + grp];
-            return make_float4(v.x * k * g.x, v.y * k * g.y, v.z * k * g.z, v.w * k * g.w);
+        float4 own[R];                                         // the block's rows, fetched before any of them is used
+#pragma unroll
+        for (int k = 0; k < R; ++k)
+            own[k] = k < nr ? *reinterpret_cast<const float4*>(x + (size_t)(r0 + k) * hidden + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        auto scaled = [&](const float4& v, int local) {
+            const float k = inv[local * groups + grp];
+            return make_float4(rounded3(v.x, k, g.x), rounded3(v.y, k, g.y), rounded3(v.z, k, g.z), rounded3(v.w, k, g.w));
         };
         float4 hist[BACK];                                     // the rows ahead, oldest first
-        int slot = row_slot[r0];
+        const int slot = row_slot[r0];
 #pragma unroll
         for (int i = 0; i < BACK; ++i) {
             const int back = BACK - i;
-            if (back <= before) hist[i] = normed(r0 - back);
+            if (back <= before) hist[i] = scaled(*reinterpret_cast<const float4*>(x + (size_t)(r0 - back) * hidden + c), before - back);
             else hist[i] = *reinterpret_cast<const float4*>(state + (size_t)slot * state_stride + (size_t)(i + before) * hidden + c);
         }
-        for (int r = r0; r < r0 + nr; ++r) {
+#pragma unroll
+        for (int k = 0; k < R; ++k) {
+            if (k >= nr) break;
+            const int r = r0 + k;
             const int s = row_slot[r];
             const bool starts = r == 0 || row_slot[r - 1] != s;
             const bool ends = r + 1 == rows || row_slot[r + 1] != s;
             float* kept = state + (size_t)s * state_stride + c;
-            if (starts && r != r0) {
+            if (starts && k != 0) {
 #pragma unroll
                 for (int i = 0; i < BACK; ++i) hist[i] = *reinterpret_cast<const float4*>(kept + (size_t)i * hidden);
             }
-            const float4 h = normed(r);
+            const float4 h = scaled(own[k], before + k);
             float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
             for (int i = 0; i < BACK; ++i) {
@@ -204,7 +234,7 @@ group_norm_conv_kernel(const float* __restrict__ x, const TG* __restrict__ gain,
         for (int j = 0; j < taps; ++j) {
             const int back = back_rows - j;
             float v;
-            if (back <= before) v = x[(size_t)(row - back) * hidden + c] * inv[j * groups + grp] * g;
+            if (back <= before) v = rounded3(x[(size_t)(row - back) * hidden + c], inv[j * groups + grp], g);
             else v = kept[(size_t)(j + before) * hidden];
             a = fmaf(taps_w[(size_t)c * taps + j], v, a);
             h = v;                                             // the last one is the row itself
@@ -220,7 +250,7 @@ group_norm_conv_kernel(const float* __restrict__ x, const TG* __restrict__ gain,
 
 // Sequences of several new tokens: the last taps - 1 rows h (older ones move up where the step brought fewer).
 template <typename TG, bool VEC>
-__global__ void __launch_bounds__(kNormThreads)
+__global__ void __launch_bounds__(kWideThreads)
 group_norm_keep_kernel(const float* __restrict__ x, const TG* __restrict__ gain, int taps, float* __restrict__ state,
                        size_t state_stride, const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_slot, int hidden,
                        int groups, float eps) {
@@ -235,11 +265,27 @@ group_norm_keep_kernel(const float* __restrict__ x, const TG* __restrict__ gain,
     const int fresh = min(n, keep), old = keep - fresh;
     inverse_roots<VEC>(x, hidden, groups, eps, fresh, sm, inv, [&](int r) { return end - fresh + r; });
     float* base = state + (size_t)seq_slot[blockIdx.x] * state_stride;
+    if constexpr (VEC) {
+        for (int c = threadIdx.x * 4; c < hidden; c += blockDim.x * 4) {
+            const float4 g = get4(gain + c);
+            for (int i = 0; i < old; ++i)
+                *reinterpret_cast<float4*>(base + (size_t)i * hidden + c) = *reinterpret_cast<const float4*>(base + (size_t)(i + fresh) * hidden + c);
+#pragma unroll 4
+            for (int i = 0; i < fresh; ++i) {
+                const float4 v = *reinterpret_cast<const float4*>(x + (size_t)(end - fresh + i) * hidden + c);
+                const float k = inv[i * groups + c / part];
+                *reinterpret_cast<float4*>(base + (size_t)(old + i) * hidden + c) =
+                    make_float4(rounded3(v.x, k, g.x), rounded3(v.y, k, g.y), rounded3(v.z, k, g.z), rounded3(v.w, k, g.w));
+            }
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
         const float g = ldf(gain, c);
         for (int i = 0; i < old; ++i) base[(size_t)i * hidden + c] = base[(size_t)(i + fresh) * hidden + c];
         for (int i = 0; i < fresh; ++i)
-            base[(size_t)(old + i) * hidden + c] = x[(size_t)(end - fresh + i) * hidden + c] * inv[i * groups + c / part] * g;
+            base[(size_t)(old + i) * hidden + c] = 
+                rounded3(x[(size_t)(end - fresh + i) * hidden + c], inv[i * groups + c / part], g);
     }
 }
 
@@ -256,6 +302,10 @@ static bool group_shape_ok(const char* what, int hidden, int groups, int rows_at
 }
 static size_t group_smem(int hidden, int groups, int rows) {
     return (size_t)rows * groups * (pieces_of(hidden / groups) + 1) * sizeof(float);
+}
+static int wide_threads(int hidden) {
+    const int t = (hidden / 4 + 31) / 32 * 32;
+    return t < 64 ? 64 : (t > kWideThreads ? kWideThreads : t);
 }
 static bool group_vec_ok(int hidden, int groups, const void* a, const void* b, const void* c, const void* d) {
     return (hidden / groups) % 4 == 0 && (((uintptr_t)a | (uintptr_t)b | (uintptr_t)c | (uintptr_t)d) & 15u) == 0;
@@ -290,22 +340,20 @@ extern "C" int citlali_group_norm_conv(const float* x, const void* gain, int gai
         return kBadShape;
     }
     // rows a block takes: several where the step has many (the rows ahead are normed once more by every block)
-    const int R = rows > 2 * device_sm_count() ? 8 : 1;
-    if (!group_shape_ok("group_norm_conv", hidden, groups, (R > taps ? R : taps) + taps)) return kBadShape;
+    const bool many = rows > 4 * device_sm_count();
+    if (!group_shape_ok("group_norm_conv", hidden, groups, 8 + taps)) return kBadShape;
     const bool vec = taps >= 2 && taps <= 4 && group_vec_ok(hidden, groups, x, gain, h_out, c_out) && ((uintptr_t)taps_w & 15u) == 0 &&
                      ((uintptr_t)state & 15u) == 0 && state_stride % 4 == 0;
     const int code = CITLALI_DISPATCH_FLOAT(gain_dtype, TG, [&] {
         return CITLALI_DISPATCH_FLOAT(out_dtype, TO, [&] {
             if (vec) {
-                const int grid = (rows + R - 1) / R;
-                const size_t smem = group_smem(hidden, groups, R + taps - 1);
-auto go = [&](auto kernel) {
-                    launch_kernel(kernel, grid, kNormThreads, smem, stream, x, (const TG*)gain, taps_w, state, state_stride, row_slot,
-                                  (TO*)h_out, (TO*)c_out, rows, hidden, groups, eps, R);
+                auto go = [&](auto kernel, int R) {
+                    launch_kernel(kernel, (rows + R - 1) / R, R == 1 ? wide_threads(hidden) : kNormThreads, group_smem(hidden, groups, R + taps - 1), stream, x, (const TG*)gain,
+                                  taps_w, state, state_stride, row_slot, (TO*)h_out, (TO*)c_out, rows, hidden, groups, eps);
                 };
-                if (taps == 2) go(group_norm_conv_vec_kernel<TG, TO, 2>);
-                else if (taps == 3) go(group_norm_conv_vec_kernel<TG, TO, 3>);
-                else go(group_norm_conv_vec_kernel<TG, TO, 4>);
+                if (taps == 2) many ? go(group_norm_conv_vec_kernel<TG, TO, 2, 8>, 8) : go(group_norm_conv_vec_kernel<TG, TO, 2, 1>, 1);
+                else if (taps == 3) many ? go(group_norm_conv_vec_kernel<TG, TO, 3, 8>, 8) : go(group_norm_conv_vec_kernel<TG, TO, 3, 1>, 1);
+                else many ? go(group_norm_conv_vec_kernel<TG, TO, 4, 8>, 8) : go(group_norm_conv_vec_kernel<TG, TO, 4, 1>, 1);
             } else {
                 launch_kernel(group_norm_conv_kernel<TG, TO>, rows, kNormThreads, group_smem(hidden, groups, taps), stream, x, (const TG*)gain,
                               taps_w, taps, state, state_stride, row_slot, (TO*)h_out, (TO*)c_out, rows, hidden, groups, eps);
@@ -316,7 +364,7 @@ auto go = [&](auto kernel) {
     if (code != 0 || taps == 1 || single_tokens) return code;
     const size_t smem = group_smem(hidden, groups, taps - 1);
     return CITLALI_DISPATCH_FLOAT(gain_dtype, TG, [&] {
-        if (vec) launch_kernel(group_norm_keep_kernel<TG, true>, sequences, kNormThreads, smem, stream, x, (const TG*)gain, taps, state, state_stride, seq_start, seq_slot, hidden, groups, eps);
+        if (vec) launch_kernel(group_norm_keep_kernel<TG, true>, sequences, wide_threads(hidden), smem, stream, x, (const TG*)gain, taps, state, state_stride, seq_start, seq_slot, hidden, groups, eps);
         else launch_kernel(group_norm_keep_kernel<TG, false>, sequences, kNormThreads, smem, stream, x, (const TG*)gain, taps, state, state_stride, seq_start, seq_slot, hidden, groups, eps);
         return CITLALI_LAUNCH_CHECK();
     });

@@ -53,7 +53,7 @@ template <typename T, typename TQ, int N>
 __global__ void __launch_bounds__(512)
 heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool, TQ* __restrict__ q_out) {
     extern __shared__ float2 trig[];                          // [rot_dims / 2] of q and k, then [vd / 2] of v
-    __shared__ float scratch[32];
+    __shared__ float2 scratch[32];
     dependents_may_launch();
     wait_for_predecessor();
     const int row = blockIdx.x, pos = a.row_pos[row], slot = a.row_slot[row];
@@ -70,6 +70,7 @@ heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool
     float q_inv = 1.0f, k_inv = 1.0f;
     if (a.q_gain) {
         float sq = 0.0f, sk = 0.0f;
+#pragma unroll 4
         for (int c = threadIdx.x * N; c < Cq + Ck; c += blockDim.x * N) {
             float v[N], b[N];
             get<N>(x + c, v);
@@ -83,8 +84,14 @@ heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool
             for (int e = 0; e < N; ++e) s = fmaf(v[e], v[e], s);
             if (c < Cq) sq += s; else sk += s;
         }
-        q_inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)Cq + a.eps);
-        k_inv = 1.0f / sqrtf(block_sum(sk, scratch) / (float)Ck + a.eps);
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) scratch[warp] = make_float2(sq, sk);
+        __syncthreads();
+        const float2 part = lane < (blockDim.x >> 5) ? scratch[lane] : make_float2(0.0f, 0.0f);
+        q_inv = 1.0f / sqrtf(warp_sum(part.x) / (float)Cq + a.eps);
+        k_inv = 1.0f / sqrtf(warp_sum(part.y) / (float)Ck + a.eps);
     }
     __syncthreads();                                          // the table of cosines and sines is complete
     const int page = a.page_table[(size_t)slot * a.table_stride + pos / a.page_size];

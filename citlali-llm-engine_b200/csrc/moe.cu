@@ -18,6 +18,8 @@ namespace citlali {
 
 constexpr int kMaxExpertsPerLane = 16;      // E <= 512
 
+// PER: experts (and groups) a lane holds at most.
+template <int PER>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, int32_t* __restrict__ chosen, int rows, int E,
                  int groups, int keep, int top, float weight_scale, int score_kind, int stride, const float* __restrict__ bias,
@@ -28,59 +30,59 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
     if (row >= rows) return;
     const float* z = logits + (size_t)row * stride;
     if (extra && lane == 0) extra[row] = 1.0f / (1.0f + expf(-z[E]));
-    float s[kMaxExpertsPerLane];
+    float s[PER];
     float m = -INFINITY;
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
         const int e = lane + 32 * j;
         s[j] = e < E ? z[e] + (bias ? bias[e] : 0.0f) : -INFINITY;
         m = fmaxf(m, s[j]);
     }
     if (score_kind == 1) {
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) s[j] = lane + 32 * j < E ? 1.0f / (1.0f + expf(-s[j])) : 0.0f;
+        for (int j = 0; j < PER; ++j) s[j] = lane + 32 * j < E ? 1.0f / (1.0f + expf(-s[j])) : 0.0f;
     } else if (score_kind == 0) {
         m = warp_max(m);
         float sum = 0.0f;
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+        for (int j = 0; j < PER; ++j) {
             const int e = lane + 32 * j;
             s[j] = e < E ? expf(s[j] - m) : 0.0f;
             sum += s[j];
         }
         sum = warp_sum(sum);
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) s[j] = s[j] / sum;
+        for (int j = 0; j < PER; ++j) s[j] = s[j] / sum;
     }
     // which experts may be chosen: bit j of `open` for expert lane + 32 j
     unsigned open = 0;
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j)
+    for (int j = 0; j < PER; ++j)
         if (lane + 32 * j < E) open |= 1u << j;
     if (groups > 1 && keep < groups) {
         const int per = E / groups;
         unsigned kept_mine = 0;                              // groups are looked at one after another; `keep` rounds
         // a group's score: the largest score in it.  Lane l keeps the scores of groups l, l + 32, ... (at most 16 each).
-        float gs[kMaxExpertsPerLane];
+        float gs[PER];
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) gs[j] = -INFINITY;
+        for (int j = 0; j < PER; ++j) gs[j] = -INFINITY;
         for (int grp = 0; grp < groups; ++grp) {
             float best = -INFINITY;
 #pragma unroll
-            for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+            for (int j = 0; j < PER; ++j) {
                 const int e = lane + 32 * j;
                 if (e < E && e / per == grp) best = fmaxf(best, s[j]);
             }
             best = warp_max(best);
 #pragma unroll
-            for (int j = 0; j < kMaxExpertsPerLane; ++j)
+            for (int j = 0; j < PER; ++j)
                 if (grp == lane + 32 * j) gs[j] = best;
         }
         for (int round = 0; round < keep; ++round) {
             float best = -INFINITY;
             int arg = 0x7fffffff;
 #pragma unroll
-            for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+            for (int j = 0; j < PER; ++j) {
                 const int grp = lane + 32 * j;
                 if (grp < groups && !(kept_mine >> j & 1u) && (gs[j] > best || (gs[j] == best && grp < arg))) { best = gs[j]; arg = grp; }
             }
@@ -91,13 +93,13 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
                 if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
             }
 #pragma unroll
-            for (int j = 0; j < kMaxExpertsPerLane; ++j)
+            for (int j = 0; j < PER; ++j)
                 if (arg == lane + 32 * j) kept_mine |= 1u << j;
         }
         // an expert is open if its group was kept: ask the lane that holds the group's bit
         unsigned allowed = 0;
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+        for (int j = 0; j < PER; ++j) {
             const int e = lane + 32 * j;
             const int grp = e < E ? e / per : 0;
             const unsigned bits = __shfl_sync(0xffffffffu, kept_mine, grp & 31);
@@ -110,7 +112,7 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
         float best = -INFINITY;
         int arg = 0x7fffffff;
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+        for (int j = 0; j < PER; ++j) {
             const int e = lane + 32 * j;
             if ((open >> j & 1u) && !(taken >> j & 1u) && (s[j] > best || (s[j] == best && e < arg))) { best = s[j]; arg = e; }
         }
@@ -121,27 +123,27 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j)
+        for (int j = 0; j < PER; ++j)
             if (arg == lane + 32 * j) taken |= 1u << j;
         if (lane == 0 && chosen) chosen[(size_t)row * top + round] = arg;
     }
     if (score_kind == 2) {                                   // softmax over the chosen logits
         float best = -INFINITY, sum = 0.0f;
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j)
+        for (int j = 0; j < PER; ++j)
             if (taken >> j & 1u) best = fmaxf(best, s[j]);
         best = warp_max(best);
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+        for (int j = 0; j < PER; ++j) {
             s[j] = (taken >> j & 1u) ? expf(s[j] - best) : 0.0f;
             sum += s[j];
         }
         sum = warp_sum(sum);
 #pragma unroll
-        for (int j = 0; j < kMaxExpertsPerLane; ++j) s[j] = s[j] / sum;
+        for (int j = 0; j < PER; ++j) s[j] = s[j] / sum;
     }
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
         const int e = lane + 32 * j;
         if (e < E) weights[(size_t)row * E + e] = (taken >> j & 1u) ? s[j] * weight_scale : 0.0f;
     }
@@ -207,8 +209,14 @@ extern "C" int citlali_moe_route(const float* logits, float* weights, int32_t* c
         set_last_error("moe_route: %d experts in %d groups of which %d are kept cannot give %d experts", E, groups, keep, top);
         return kBadShape;
     }
-    launch_kernel(moe_route_kernel, (rows + 3) / 4, 128, 0, stream, logits, weights, chosen, rows, E, groups, keep, top, weight_scale,
-                  score_kind, stride, bias, extra);
+    auto go = [&](auto kernel) {
+        launch_kernel(kernel, (rows + 3) / 4, 128, 0, stream, logits, weights, chosen, rows, E, groups, keep, top, weight_scale, score_kind,
+                      stride, bias, extra);
+    };
+    if (E <= 32) go(moe_route_kernel<1>);
+    else if (E <= 64) go(moe_route_kernel<2>);
+    else if (E <= 128) go(moe_route_kernel<4>);
+    else go(moe_route_kernel<kMaxExpertsPerLane>);
     return CITLALI_LAUNCH_CHECK();
 }
 

@@ -339,9 +339,22 @@ def _check_sink_and_turns(sink, turns, heads, rows, value_dim):
 
 
 def attention_prefill_tc(q, q_stride, k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, sequences, max_new,
-                         nq, nkv, head_dim, page_size, window, scale, error_flag=None):
-    """Prompt attention on tcgen05 (head size 128, pages of 64)."""
-    _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, error_flag)
+                         nq, nkv, head_dim, page_size, window, scale, error_flag=None, softcap=0.0, gate=None, sink=None,
+                         turns=None, turn_pairs=False):
+    """Prompt attention on tcgen05 (head size 128, pages of 64).  ``softcap``, ``gate``, ``sink``, ``turns``, ``turn_pairs``: see
+    :func:`attention_prefill`."""
+    _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, error_flag, sink, turns)
+    if softcap or gate is not None or sink is not None or turns is not None:
+        require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
+                "attention_prefill_tc: bfloat16 only")
+        _check_sink_and_turns(sink, turns, nq, out.shape[0], head_dim)
+        _check(lib().citlali_attention_prefill_tc_with(
+            _ptr(q), _i(q_stride), _i(q.shape[0]), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(page_table),
+            _i(page_table.shape[1]), _ptr(seq_start), _ptr(seq_slot), _ptr(seq_past), _ptr(out), _i(out.shape[1]),
+            _i(sequences), _i(max_new), _i(nq), _i(nkv), _i(head_dim), _i(page_size), _i(window or 0), _f(scale),
+            _ptr(error_flag), _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink),
+            _ptr(turns), _i(1 if turn_pairs else 0), _stream()), "attention_prefill_tc")
+        return
     require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
             "attention_prefill_tc: bfloat16 only")
     _check(lib().citlali_attention_prefill_tc(
@@ -371,6 +384,29 @@ def attention_decode(q, q_stride, k_pool, v_pool, page_table, row_slot, row_pos,
         # one kernel whose blocks merge through distributed shared memory, or a partial and a merge kernel
         "attention_decode" if (page_size == 64 and q_stride % 8 == 0 and q.data_ptr() % 16 == 0
                                and head_dim in (16, 32, 48, 64, 80, 96, 112, 128, 256)) else "attention_decode_merged")
+
+
+def attention_decode_with(q, kv, batch, out, nq, nkv, d, vd, window, scale, softcap=0.0, gate=None, sink=None, turns=None,
+                          turn_pairs=False):
+    """Split-context attention of single tokens on the tensor cores with a value size of its own, a soft cap, a gate, sinks and
+    turned-back outputs (see :func:`attention_prefill`)."""
+    _need_cuda(q, kv.keys, kv.values, kv.page_table, out, sink, turns)
+    rows = out.shape[0]
+    require(q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+            and q.shape == (rows, nq * d) and out.shape == (rows, nq * vd), "attention_decode_with: shapes or dtypes do not fit")
+    _check_sink_and_turns(sink, turns, nq, rows, vd)
+    l = lib()
+    l.citlali_attention_decode_scratch_floats.restype = ctypes.c_size_t
+    positions = kv.page_table.shape[1] * kv.page_size
+    need = l.citlali_attention_decode_scratch_floats(_i(rows), _i(nq), _i(max(d, vd)), _i(kv.page_size), _i(positions))
+    ws = _scratch(q.device, "attention_decode", need * 4)
+    counters = _scratch(q.device, "attention_decode counters", rows * nq * 4, zeroed=True)
+    _check(l.citlali_attention_decode_with(
+        _ptr(q), _i(q.shape[1]), _ptr(kv.keys), _ptr(kv.values), _ptr(kv.page_table), _i(kv.page_table.shape[1]),
+        _ptr(batch.row_slot), _ptr(batch.row_pos), _ptr(out), _i(out.shape[1]), _ptr(ws), _sz(ws.numel() // 4), _ptr(counters),
+        _sz(counters.numel() // 4), _i(rows), _i(nq), _i(nkv), _i(d), _i(vd), _i(kv.page_size), _i(int(window or 0)), _f(scale),
+        _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink), _ptr(turns),
+        _i(1 if turn_pairs else 0), _stream()), "attention_decode_with")
 
 
 _sm_count = {}
@@ -835,10 +871,11 @@ def heads_prepare(proj, batch, kv, q_out, nq, nkv, d, vd, bias=None, q_gain=None
 
 
 def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scale, softcap=0.0, gate=None, sink=None,
-                     turns=None, turn_pairs=False):
-    """Attention of every row over its slot's cache, through a window that keeps the first tokens.  bfloat16 steps that
-    bring runs of tokens, with keys and values of sizes the tensor-core kernel takes, run that kernel; steps of single
-    tokens, the 32-bit path and other sizes run the kernel whose launch depends on the row count alone.  ``softcap`` c > 0:
+                     turns=None, turn_pairs=False, error_flag=None):
+    """Attention of every row over its slot's cache, through a window that keeps the first tokens.  bfloat16 steps with keys
+    and values of sizes the tensor-core kernels take run those: the split-context kernel where every sequence brings one
+    token (and no first tokens are kept), the prompt kernel otherwise; the 32-bit path and other sizes run the kernel whose
+    launch depends on the row count alone.  ``softcap`` c > 0:
     the scaled scores become c tanh(s / c).  ``sink``, ``turns``, ``turn_pairs``: see :func:`attention_prefill`.  ``gate``: float32 columns of a matrix (a view whose rows may be further apart
     than they are long), the output is multiplied by their sigmoids element by element."""
     _need_cuda(q, kv.keys, kv.values, kv.page_table, out, sink, turns)
@@ -854,11 +891,25 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
     softcap = float(softcap or 0.0)
     if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and not batch.is_decode
             and (nq * d) % 8 == 0 and not torch.cuda.is_current_stream_capturing()
+            and (gate is None or (gate_stride % 4 == 0 and gate.data_ptr() % 16 == 0))
+            and d == vd and batch.max_new >= 48 and not (window and keep_first)
+            and lib().citlali_attention_prefill_tc_supports(_i(d), _i(kv.page_size))):
+        attention_prefill_tc(q, nq * d, kv.keys, kv.values, kv.page_table, batch.seq_start, batch.seq_slot, batch.seq_past, out,
+                             batch.sequences, batch.max_new, nq, nkv, d, kv.page_size, window, scale, error_flag, softcap=softcap,
+                             gate=gate, sink=sink, turns=turns, turn_pairs=turn_pairs)
+        return
+    if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and not batch.is_decode
+            and (nq * d) % 8 == 0 and not torch.cuda.is_current_stream_capturing()
             and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 8 == 0))
             and lib().citlali_attention_prefill_supports_sizes(_i(d), _i(vd), _i(kv.page_size))):
         attention_prefill(q, nq * d, kv.keys, kv.values, kv.page_table, batch.seq_start, batch.seq_slot, batch.seq_past, out,
                           batch.sequences, batch.max_new, nq, nkv, d, kv.page_size, window, scale, keep_first=keep_first,
                           softcap=softcap, gate=gate, value_dim=vd, sink=sink, turns=turns, turn_pairs=turn_pairs)
+        return
+    if (batch.is_decode and q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and (nq * d) % 8 == 0
+            and not (window and keep_first) and lib().citlali_attention_decode_with_supports(_i(d), _i(vd), _i(kv.page_size))):
+        attention_decode_with(q, kv, batch, out, nq, nkv, d, vd, window, scale, softcap=softcap, gate=gate, sink=sink,
+                              turns=turns, turn_pairs=turn_pairs)
         return
     longest = kv.page_table.shape[1] * kv.page_size          # a bound that no step's lengths change
     max_keys = min(longest, window + keep_first) if window else longest

@@ -152,6 +152,7 @@ class WindowAttention:
         elif self.sink is not None:
             self.sinks = torch.full((self.nq,), float(self.sink), dtype=torch.float32, device=ctx.device)
         self.dtype = ctx.dtype
+        self.error_flag = ctx.error_flag
 
     def forward(self, h, batch, cache_view, residual, write_cache=True, overwrite=False):
         require(isinstance(cache_view, tuple) and len(cache_view) == (2 if self.taps > 1 else 1),
@@ -178,7 +179,7 @@ class WindowAttention:
         out = torch.empty((rows, self.nq * self.vd), dtype=self.dtype, device=proj.device)
         ops.attention_window(q, kv, batch, out, self.nq, self.nkv, self.d, self.vd, self.window, self.keep_first, self.scale,
                              softcap=self.softcap, gate=proj[:, self.C:] if self.has_gate else None, sink=self.sinks,
-                             turns=turns, turn_pairs=self.v_layout == "pairs")
+                             turns=turns, turn_pairs=self.v_layout == "pairs", error_flag=self.error_flag)
         if overwrite:
             self.o.forward(out, out=residual)
         else:
