@@ -901,6 +901,8 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
     if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and not batch.is_decode
             and (nq * d) % 8 == 0 and not torch.cuda.is_current_stream_capturing()
             and (gate is None or (gate_stride % 2 == 0 and gate.data_ptr() % 8 == 0))
+            # (keys and values of different sizes: only where single tokens run the tensor-core kernel too, and round alike)
+            and (d == vd or not (window and keep_first))
             and lib().citlali_attention_prefill_supports_sizes(_i(d), _i(vd), _i(kv.page_size))):
         attention_prefill(q, nq * d, kv.keys, kv.values, kv.page_table, batch.seq_start, batch.seq_slot, batch.seq_past, out,
                           batch.sequences, batch.max_new, nq, nkv, d, kv.page_size, window, scale, keep_first=keep_first,
