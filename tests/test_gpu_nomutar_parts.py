@@ -57,6 +57,12 @@ MIXERS = [
     (32, mixer(C, 5, 5, 12, 20, 0.3, (4, 20.0), None)),
     (48, mixer(C, 2, 1, 256, 136, 0.06, (256, 1e6), None)),                                      # the widest tiles
     (48, mixer(C, 32, 2, 64, 64, 0.125, (64, 1e4), None)),                                       # sixteen query heads a key head
+    # heads of 128: the prompt kernel with its tiles in tensor memory, with scores under a cap that zero serves as a reference
+    # for, under one too wide for that, without a cap, and with an odd number of query heads a key head
+    (64, mixer(A, 8, 2, 128, 128, 0.09, (64, 50.0), None, softcap=20.0, window=130, scaling=wavelength(2.0, 0.5, 16.0, 4096))),
+    (32, mixer(A, 4, 2, 128, 128, 0.2, (128, 500.0), None, softcap=90.0)),
+    (32, mixer(A, 3, 1, 128, 128, 0.09, (32, 100.0), None, window=70)),
+    (40, mixer(C, 4, 2, 128, 128, 0.15, (128, 1e4), None)),
 ]
 
 
@@ -323,6 +329,40 @@ def test_residual_convolution(hidden, groups, taps, dtype):
         for g, t in zip(both[n], want[n]):
             assert bool(((g - t).abs() <= tol * (t.abs() + 1.0)).all()), n
     assert torch.equal(both["a"][1], first[1])
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("hidden,groups,taps", [(64, 4, 3), (96, 1, 2), (128, 8, 4), (60, 4, 5)])
+def test_residual_convolution_of_long_steps(hidden, groups, taps, dtype):
+    """Steps of more than a thousand rows (a block then takes several rows): one sequence, and a batch whose sequences begin and
+    end inside such a block, some of them with fewer new tokens than the convolution looks back."""
+    norm = build_part("norm", PartSpec("grouped_rms_norm", {"size": hidden, "groups": groups, "eps": 1e-3, "tensor": "n.norm1"}, "n"))
+    conv = build_part("mixer_input", PartSpec("residual_conv", {"hidden_size": hidden, "taps": taps}, "n.canon1"))
+    w = draw(norm.tensor_specs() + conv.tensor_specs(), 4)
+    ctx = ctx_for(dtype)
+    norm.bind(handles(w), ctx)
+    conv.bind(handles(w), ctx)
+    tol = 2e-6 if dtype == torch.float32 else 6e-3
+    for steps in ([[1300], [900], [1]], [[701, 1, 2, 3, 600, 1], [1, 1, 1, 1, 1, 1], [2, 640, 1, 700, 3, 5], [3, 2, 1, 1, 9, 1]]):
+        n = len(steps[0])
+        cache = cb.SequenceCache([conv.cache_requirement()], n, 64, 4096, dtype, DEV)
+        slots = [cache.acquire() for _ in range(n)]
+        total = [sum(st[i] for st in steps) for i in range(n)]
+        x = [torch.randn(t, hidden, generator=torch.Generator().manual_seed(i)).float() for i, t in enumerate(total)]
+        done, got = [0] * n, [[] for _ in range(n)]
+        for st in steps:
+            batch = pack_step([StepEntry(slots[i], [0] * st[i], []) for i in range(n)], done, 1, DEV)
+            rows = torch.cat([x[i][done[i]:done[i] + st[i]] for i in range(n)]).to(DEV).contiguous()
+            h, m = conv.forward(norm, rows, batch, cache.view(0))
+            at = 0
+            for i in range(n):
+                got[i].append(m[at:at + st[i]].double().cpu())
+                at += st[i]
+                done[i] += st[i]
+        for i in range(n):
+            h = plain.group_norm(x[i].double(), w["n.norm1"], groups, 1e-3)
+            want = h + plain.causal_conv(h, w["n.canon1"])
+            assert bool(((torch.cat(got[i]) - want).abs() <= tol * (want.abs() + 1.0)).all()), (i, steps)
 
 
 # ---- the embedding of pairs ----------------------------------------------------------------------------------------------------
