@@ -15,7 +15,7 @@ import torch
 from .. import ops
 from ..config.spec import ModelSpec
 from ..errors import require
-from ..parts.base import BuildContext, StepBatch, build_part, part_class
+from ..parts.base import BuildContext, StepBatch, build_part, named_sources, part_class
 from ..parts.linear import DenseLinear
 from ..weights.loader import TensorSpec, WeightHandle
 
@@ -120,6 +120,17 @@ class DecoderModel:
         else:
             require(spec.head_name in weights, f"missing required tensor: {spec.head_name}")
             self.head.bind(weights, ctx)
+
+    def kernel_sources(self) -> List[str]:
+        """The kernel sources the model's steps call, as far as its parts name them (``csrc/<name>.cu``)."""
+        dtype = self.ctx.dtype
+        out = {"elementwise", "gemm_simt" if dtype == torch.float32 else "gemm_tcgen05"}
+        if self.spec.residual_streams is not None:
+            out.add("hyper_connection")
+        for owner in [self.final_norm, self.embedding_norm, self.embedding_addition] + [p for b in self.layers for p in [b] + list(b.parts())]:
+            if owner is not None:
+                out.update(named_sources(owner, dtype))
+        return sorted(out)
 
     def weight_bytes_read_per_step(self) -> int:
         """Bytes of weights one step reads when each matrix it uses is read once: every tensor the layers

@@ -70,6 +70,7 @@ class InferenceSession:
             spec = config.to_model_spec()
             ctx = self._context(dev, dtype)
             model = DecoderModel(spec, ctx)
+            ops.prepare_kernels(model.kernel_sources())
             weights = loader.load_all(model.tensor_specs(), device="cpu", progress=progress)
             model.bind(weights)
         finally:
@@ -88,6 +89,7 @@ class InferenceSession:
         spec = config.to_model_spec()
         ctx = self._context(dev, dtype)
         model = DecoderModel(spec, ctx)
+        ops.prepare_kernels(model.kernel_sources())
         stored = parse_dtype(stored_dtype if stored_dtype is not None else dtype)
         handles: Dict[str, WeightHandle] = {}
         for s in model.tensor_specs():

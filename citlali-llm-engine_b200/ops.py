@@ -36,6 +36,12 @@ def lib():
     return _lib
 
 
+def prepare_kernels(sources) -> None:
+    """Compile (where stale) and load these kernel sources ahead of their first use, side by side."""
+    from .csrc.build import load
+    load().prepare(sources)
+
+
 def _ptr(t: Optional[torch.Tensor]):
     if t is None:
         return ctypes.c_void_p(0)
@@ -892,7 +898,7 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
     if (q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and not batch.is_decode
             and (nq * d) % 8 == 0 and not torch.cuda.is_current_stream_capturing()
             and (gate is None or (gate_stride % 4 == 0 and gate.data_ptr() % 16 == 0))
-            and d == vd and batch.max_new >= 48 and not (window and keep_first)
+            and d == vd == 128 and batch.max_new >= 48 and not (window and keep_first)
             and lib().citlali_attention_prefill_tc_supports(_i(d), _i(kv.page_size))):
         attention_prefill_tc(q, nq * d, kv.keys, kv.values, kv.page_table, batch.seq_start, batch.seq_slot, batch.seq_past, out,
                              batch.sequences, batch.max_new, nq, nkv, d, kv.page_size, window, scale, error_flag, softcap=softcap,

@@ -60,6 +60,11 @@ class GQAttention:
             return False
         return self.position.inv_freq is not None or bool(getattr(self.position, "graph_safe", False))
 
+    def kernel_sources(self, dtype):
+        if dtype == torch.float32:
+            return ("attention_generic",)
+        return ("attention_generic", "attention_decode", "attention_prefill") + (("attention_prefill_tc",) if self.d == 128 else ())
+
     # ---- what it needs ---------------------------------------------------------------
     def tensor_specs(self):
         specs = self.qkv.tensor_specs() + self.o.tensor_specs()

@@ -12,6 +12,9 @@ Interfaces (all tensors are on the model's device; ``x`` is the float32 residual
 * every part: ``__init__(params, prefix)`` (no device work), ``tensor_specs()`` -> the
   checkpoint tensors it needs, ``bind(weights, ctx)`` -> take them from a ``{name: WeightHandle}``
   map onto the device.
+* any part may name the kernel sources (``csrc/<name>.cu``) it is going to call, so that a first load compiles them side by
+  side: ``kernel_sources``, a tuple, or a function of the compute dtype that gives one.  What is not named is compiled when
+  it is first called.
 * norm: ``forward(x, row_index=None) -> h`` (``row_index`` int32 picks and orders rows).
 * mixer: ``cache_requirement()`` -> KVRequirement | StateRequirement | None;
   ``forward(h, batch, cache_view, residual, write_cache)`` adds its output into ``residual``
@@ -63,6 +66,12 @@ def registered_parts(role: str) -> List[str]:
 def build_part(role: str, spec):
     """The part a :class:`PartSpec` describes, from the registry of ``role``."""
     return part_class(role, spec.kind)(spec.params, spec.prefix)
+
+
+def named_sources(part, dtype) -> tuple:
+    """The kernel sources a part (or a block) names, see the module's head."""
+    named = getattr(part, "kernel_sources", ())
+    return tuple(named(dtype) if callable(named) else named)
 
 
 @dataclass

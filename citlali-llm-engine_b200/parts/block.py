@@ -101,6 +101,7 @@ class SublayerOutputNormBlock:
     the kernel that did the sum before (for a model's first layer by a conversion of its own; none in the 32-bit path, where
     the sub-layers read the residual's own memory).  Any registered mixer or feed-forward serves: one that says
     ``can_overwrite`` stores its output, any other adds it into a zeroed buffer."""
+    kernel_sources = ("sublayer",)
 
     def __init__(self, layer_spec):
         has = layer_spec.parts.__contains__
@@ -162,6 +163,7 @@ class SandwichNormBlock:
     The next sub-layer may be the next layer's: this block then leaves the normed rows for it (``StepBatch.normed_carry``:
     the rows and the norm they went through), and a block that finds rows made by its own first norm skips that norm.  A sub-layer that offers ``deferred_bias`` (its output's bias) has it added in the same kernel.
     Other norms run one by one (``forward`` in front, ``add_into`` behind)."""
+    kernel_sources = ("sublayer",)
 
     def __init__(self, layer_spec):
         has = layer_spec.parts.__contains__
@@ -281,6 +283,7 @@ class InputInjectionBlock:
     and the sum are float32.  ``block_params``: hidden_size, passes, ``matrix`` and ``steps`` (the tensors' full names)."""
     needs_embedding_output = True
     graph_safe = True
+    kernel_sources = ("activations",)
 
     def __init__(self, layer_spec):
         bp = layer_spec.block_params

@@ -50,6 +50,7 @@ def bind_float32(weights, name: str, shape, ctx) -> torch.Tensor:
 class GatedDeltaMixer:
     graph_safe = True        # slots and row ranges are read on the device; the launches depend on the counts alone
     can_overwrite = True
+    kernel_sources = ("delta_rule",)
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

@@ -66,6 +66,9 @@ class GatedSiluFeedForward:
             self.deferred_bias = bind_vector(weights, nm["down_bias"], self.hidden, ctx)
         self.dtype = ctx.dtype
 
+    def kernel_sources(self, dtype):
+        return () if self.plain else ("activations",)
+
     def can_absorb_norm(self) -> bool:
         if not self.plain:
             return False
@@ -109,6 +112,7 @@ class SquaredReluFeedForward:
     (the matrices' full names; default ``<prefix>.up_proj.weight`` and ``<prefix>.down_proj.weight``)."""
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("hyper_connection",)
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])
@@ -146,6 +150,7 @@ class XieluFeedForward:
     ``deferred_bias`` and pass ``defer_bias=True``."""
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("activations",)
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

@@ -32,6 +32,7 @@ from .norm import RMSNorm
 
 class HyperConnectionBlock:
     takes_stream_write = True        # does the write-back the block ahead left in ``batch.stream_write``
+    kernel_sources = ("hyper_connection",)
 
     def __init__(self, layer_spec):
         has = layer_spec.parts.__contains__

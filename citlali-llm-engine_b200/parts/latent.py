@@ -40,6 +40,7 @@ from .linear import DenseLinear
 class LatentAttention:
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("latent_attention", "latent_attention_mma")
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

@@ -23,6 +23,7 @@ from .delta import bind_float32
 
 class ResidualConv:
     graph_safe = True
+    kernel_sources = ("group_norm",)
 
     def __init__(self, params, prefix: str):
         self.hidden, self.taps = int(params["hidden_size"]), int(params["taps"])

@@ -43,6 +43,7 @@ from .linear import DenseLinear, ExpertDown, ExpertGateUp
 class RoutedExperts:
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("moe", "activations")
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

@@ -60,6 +60,7 @@ class RMSNorm:
 class GroupedRMSNorm(RMSNorm):
     """An RMS norm over ``groups`` equal consecutive parts of the row: every part is divided by its own
     sqrt(mean(part^2) + eps), then the whole row is multiplied by the gain (``offset + w``, as in :class:`RMSNorm`)."""
+    kernel_sources = ("group_norm",)
 
     def __init__(self, params, prefix: str):
         super().__init__(params, prefix)
@@ -86,6 +87,7 @@ class LayerNorm:
     Parameters: size, eps; optional ``tensor`` (the gain's full name; default ``<prefix>.weight``) and ``bias`` (the bias's
     full name; None: no bias).  A norm with a bias keeps gain and bias in float32 in both paths."""
     graph_safe = True
+    kernel_sources = ("sublayer",)
 
     def __init__(self, params, prefix: str):
         self.size = int(params["size"])

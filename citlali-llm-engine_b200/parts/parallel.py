@@ -12,7 +12,7 @@ import torch
 from .. import ops
 from ..config.spec import PartSpec
 from ..errors import require
-from .base import build_part, register_part
+from .base import build_part, named_sources, register_part
 
 
 def _spec(d) -> PartSpec:
@@ -32,6 +32,9 @@ class ParallelMixers:
     @property
     def graph_safe(self) -> bool:
         return bool(getattr(self.left, "graph_safe", False)) and bool(getattr(self.right, "graph_safe", False))
+
+    def kernel_sources(self, dtype):
+        return ("sublayer",) + named_sources(self.left, dtype) + named_sources(self.right, dtype)
 
     def tensor_specs(self):
         return self.left.tensor_specs() + self.right.tensor_specs()

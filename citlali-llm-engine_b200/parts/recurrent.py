@@ -32,6 +32,7 @@ _ROLES = ("y", "y_bias", "x", "x_bias", "conv", "conv_bias", "gate_a", "gate_a_b
 class GatedRecurrentMixer:
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("recurrent",)
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

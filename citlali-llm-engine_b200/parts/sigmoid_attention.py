@@ -47,6 +47,7 @@ _DEFAULTS = {"q": "q", "k": "k", "v": "v", "o": "o", "talk": "talk", "head_bias"
 
 class SigmoidAttention:
     can_overwrite = True
+    kernel_sources = ("sigmoid_attention", "sigmoid_attention_mma", "activations")
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

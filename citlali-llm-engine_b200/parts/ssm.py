@@ -33,6 +33,7 @@ from .linear import DenseLinear
 class StateSpaceMixer:
     graph_safe = True
     can_overwrite = True
+    kernel_sources = ("delta_rule", "recurrent")
 
     def __init__(self, params, prefix: str):
         self.hidden = int(params["hidden_size"])

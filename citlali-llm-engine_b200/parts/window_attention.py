@@ -116,6 +116,13 @@ class WindowAttention:
             specs += [TensorSpec(nm[r + "_bias"], (size,), "state") for r, size in zip(("q", "k", "v"), self.sizes)]
         return specs
 
+    def kernel_sources(self, dtype):
+        prepared = ("heads_prepare",) if self.plain_heads else ("window_attention",)
+        kept = ("recurrent",) if self.taps > 1 else ()
+        if dtype == torch.float32 or self.d % 8 or self.vd % 8 or self.keep_first:
+            return prepared + kept + ("window_attention",)
+        return prepared + kept + ("attention_decode", "attention_prefill") + (("attention_prefill_tc",) if self.d == self.vd == 128 else ())
+
     def norm_sizes(self):
         return (self.nq * self.d, self.nkv * self.d) if self.norm_whole else (self.d, self.d)
 

@@ -6,7 +6,7 @@ import subprocess
 
 import pytest
 
-from citlali_b200 import ops
+from citlali_b200.csrc import build as kernel_build
 
 pytestmark = pytest.mark.gpu
 HERE = os.path.dirname(os.path.abspath(__file__))
@@ -16,7 +16,7 @@ def test_a_cpp_program_calls_the_kernels_through_the_c_interface(tmp_path):
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(nvcc):
         pytest.skip("no nvcc to build the example with")
-    ops.lib()                                                   # makes sure the library is built
+    kernel_build.build()                                        # the whole library, if it is not there yet
     csrc = os.path.join(os.path.dirname(HERE), "citlali-llm-engine_b200", "csrc")
     lib_dir = os.path.join(csrc, "_build")
     exe = str(tmp_path / "abi_example")
