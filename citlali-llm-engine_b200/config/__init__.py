@@ -10,6 +10,8 @@ from .pivavik import PivavikConfig
 from . import pivavik as _pivavik
 from .nomutar import NomutarConfig
 from . import nomutar as _nomutar
+from .kopalorn import KopalornConfig
+from . import kopalorn as _kopalorn
 from .registry import (config_class_for, config_from_dict, config_from_model_dir,
                        register_architecture, registered_architectures, unregister_architecture)
 
@@ -19,3 +21,4 @@ register_architecture(_gidirax.ARCHITECTURE, GidiraxConfig)
 register_architecture(_sobunex.ARCHITECTURE, SobunexConfig)
 register_architecture(_pivavik.ARCHITECTURE, PivavikConfig)
 register_architecture(_nomutar.ARCHITECTURE, NomutarConfig)
+register_architecture(_kopalorn.ARCHITECTURE, KopalornConfig)

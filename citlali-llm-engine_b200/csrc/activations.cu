@@ -13,6 +13,8 @@
 //                     not read), or, with weight_input, of the activation of gate and up each times that weight (the
 //                     expert applied to its weighted input).  The expert for every row comes last, has a width, run and
 //                     limit of its own and weight 1, or a weight a row of its own (tail_weights).
+//   expert_relu_squared  the activation of experts without a gate: weights[r, e] max(z, 0)^2 over z [rows, E ff], a zero weight
+//                     giving zeros; behind them an expert that every row uses, with a width and a weight a row of its own.
 #include "api.h"
 #include "common.cuh"
 
@@ -158,6 +160,33 @@ expert_gate_vec_kernel(const TZ* __restrict__ gu, const float* __restrict__ weig
     }
 }
 
+template <typename TZ, typename TO, bool VEC>
+__global__ void __launch_bounds__(256)
+expert_relu_squared_kernel(const TZ* __restrict__ z, const float* __restrict__ weights, TO* __restrict__ act, int E, int ff,
+                           int tail_ff, const float* __restrict__ tail_weights) {
+    dependents_may_launch();
+    wait_for_predecessor();
+    const int row = blockIdx.x, routed = E * ff, n = routed + tail_ff;
+    const TZ* in = z + (size_t)row * n;
+    TO* o = act + (size_t)row * n;
+    constexpr int W = VEC ? 4 : 1;                            // (widths are multiples of four: a piece lies within one expert)
+    auto squared = [](float u) { u = fmaxf(u, 0.0f); return u * u; };
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * W; i < n; i += gridDim.y * blockDim.x * W) {
+        const bool tail = i >= routed;
+        const float w = tail ? (tail_weights ? tail_weights[row] : 1.0f) : weights[(size_t)row * E + i / ff];
+        if constexpr (VEC) {
+            float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (w != 0.0f) {
+                const float4 u = load4(in + i);
+                r = make_float4(w * squared(u.x), w * squared(u.y), w * squared(u.z), w * squared(u.w));
+            }
+            store4(o + i, r);
+        } else {
+            stf(o, i, w != 0.0f ? w * squared(ldf(in, i)) : 0.0f);
+        }
+    }
+}
+
 }  // namespace citlali
 
 using namespace citlali;
@@ -216,6 +245,26 @@ extern "C" int citlali_expert_gate(const void* gate_up, int in_dtype, const floa
             launch_kernel(expert_gate_kernel<TZ, TO>, grid, 256, 0, stream, (const TZ*)gate_up, weights, (TO*)act, E, ff,
                           run > 0 ? run : 1, kind, limit, alpha, tail_ff, tail_run > 0 ? tail_run : 1, tail_limit, bias, weight_input,
                           tail_weights);
+            return CITLALI_LAUNCH_CHECK();
+        });
+    });
+}
+
+extern "C" int citlali_expert_relu_squared(const void* z, int z_dtype, const float* weights, void* act, int act_dtype, int rows, int E,
+                                           int ff, int tail_ff, const float* tail_weights, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (E < 0 || ff < 0 || tail_ff < 0 || (E > 0 && (ff <= 0 || weights == nullptr)) || E * ff + tail_ff <= 0) {
+        set_last_error("expert_relu_squared: %d experts of %d, an expert for all of %d", E, ff, tail_ff);
+        return kBadShape;
+    }
+    const int n = E * ff + tail_ff;
+    const bool vec = (E == 0 || ff % 4 == 0) && tail_ff % 4 == 0 && (((uintptr_t)z | (uintptr_t)act) & 15u) == 0;
+    const int by = ((vec ? n / 4 : n) + 255) / 256;
+    const dim3 grid(rows, by < 64 ? by : 64);
+    return CITLALI_DISPATCH_FLOAT(z_dtype, TZ, [&] {
+        return CITLALI_DISPATCH_FLOAT(act_dtype, TO, [&] {
+            if (vec) launch_kernel(expert_relu_squared_kernel<TZ, TO, true>, grid, 256, 0, stream, (const TZ*)z, weights, (TO*)act, E, E > 0 ? ff : 1, tail_ff, tail_weights);
+            else launch_kernel(expert_relu_squared_kernel<TZ, TO, false>, grid, 256, 0, stream, (const TZ*)z, weights, (TO*)act, E, E > 0 ? ff : 1, tail_ff, tail_weights);
             return CITLALI_LAUNCH_CHECK();
         });
     });

@@ -112,7 +112,7 @@ int citlali_attention_decode_with(const void* q, int q_stride, const void* k_poo
                                   int out_stride, float* partial, size_t partial_floats, int32_t* counters, size_t counter_ints,
                                   int rows, int nq, int nkv, int head_dim, int value_dim, int page_size, int window, float scale,
                                   float softcap, const float* gate, size_t gate_stride, const float* sink, const float* turns,
-                                  int turn_pairs, cudaStream_t stream);
+                                  int turn_pairs, float* out32, cudaStream_t stream);
 void citlali_attention_decode_set_split(int split);
 void citlali_attention_decode_set_by_length(int on, int run_scale_q8);
 void citlali_attention_decode_set_per_warp(int on);
@@ -127,10 +127,11 @@ int citlali_attention_prefill(const void* q, int q_stride, const void* k_pool, c
                               void* out, int out_stride, int sequences, int max_new,
                               int nq, int nkv, int head_dim, int value_dim, int page_size, int window, int keep_first,
                               float scale, float softcap, const float* gate, size_t gate_stride, const float* sink,
-                              const float* turns, int turn_pairs, cudaStream_t stream);
+                              const float* turns, int turn_pairs, float* out32, cudaStream_t stream);
 // sink [nq] (may be null): the softmax's denominator also counts exp(sink[head]), neither scaled nor capped.  turns
 // [rows, value_dim / 2] (cos, sin) (may be null; 16-byte aligned): the result's pairs (m, m + value_dim / 2), or with
-// turn_pairs (2m, 2m + 1), are turned back by the row's angles, ahead of the gate.  Keys and values of different sizes:
+// turn_pairs (2m, 2m + 1), are turned back by the row's angles, ahead of the gate.  out32 (may be null; not with turns): the
+// result goes there in float32, rows out_stride apart, and out is not written.  Keys and values of different sizes:
 int citlali_attention_prefill_supports_sizes(int head_dim, int value_dim, int page_size);
 
 // The same on tcgen05 (scores and output in tensor memory), for head size 128 and pages of 64.
@@ -149,7 +150,7 @@ int citlali_attention_prefill_tc_with(const void* q, int q_stride, int total_row
                                       const int32_t* seq_slot, const int32_t* seq_past, void* out, int out_stride, int sequences,
                                       int max_new, int nq, int nkv, int head_dim, int page_size, int window, float scale,
                                       int32_t* error_flag, float softcap, const float* gate, size_t gate_stride, const float* sink,
-                                      const float* turns, int turn_pairs, cudaStream_t stream);
+                                      const float* turns, int turn_pairs, float* out32, cudaStream_t stream);
 
 // tokens[r] = argmax of logits[r, :] over finite values, lowest index on ties.
 int citlali_argmax_rows(const float* logits, int32_t* tokens, int rows, int vocab, cudaStream_t stream);
@@ -259,6 +260,13 @@ int citlali_layer_norm_rows(const float* x, const void* gain, const void* bias, 
 int citlali_layer_norm_chain(const float* y, const float* in_bias, const float* g1, const float* b1, float* x, void* emit,
                              const float* g2, const float* b2, void* out2, int out_dtype, int rows, int hidden, float eps1,
                              float eps2, cudaStream_t stream);
+// x[r] += x0[r] (may be null) + step; with gain also out[r] = layer_norm(x[r]) * gain + bias in out_dtype (float32 vectors; bias
+// may be null).
+int citlali_add_rows_norm(float* x, const float* x0, const float* step, const float* gain, const float* bias, void* out,
+                          int out_dtype, int rows, int hidden, float eps, cudaStream_t stream);
+// out[r] = a rms(l[r]) wl + b rms(r[r]) wr over float32 rows, rms(v) = v / sqrt(mean(v^2) + eps); out may be l or r.
+int citlali_normed_pair_sum(float a, const float* l, const float* wl, float b, const float* r, const float* wr, float* out,
+                            int rows, int hidden, float eps_l, float eps_r, cudaStream_t stream);
 // out = x converted from float32.
 int citlali_cast_rows(const float* x, void* out, int out_dtype, size_t n, cudaStream_t stream);
 // out = a l + b r over n floats.
@@ -299,6 +307,28 @@ int citlali_gated_scan(const float* a, const float* coef, const float* side, int
                        float* state, size_t state_stride, size_t state_off, const int32_t* seq_start, const int32_t* seq_slot,
                        int sequences, void* out, int out_dtype, int width, cudaStream_t stream);
 
+// ---- memories that are decayed sums of outer products ---------------------------------------------------------------
+// Log gates with a running maximum: i = cap tanh((zi + bi) / cap), f = logsigmoid(cap tanh((zf + bf) / cap)), m_t =
+// max(f + m_(t-1), i) from and into state[slot][max_off + h]; logs [rows, H, 2] = (f + m_(t-1) - m_t, i - m_t), floors
+// [rows, H] = exp(-m_t).  zi, zf: a head's first columns, rows `stride` floats apart; bi, bf [H] (may be null).
+int citlali_memory_gates(const float* zi, const float* zf, size_t stride, const float* bi, const float* bf, float cap,
+                         float* state, size_t state_stride, size_t max_off, const int32_t* seq_start, const int32_t* seq_slot,
+                         int sequences, int H, float* logs, float* floors, cudaStream_t stream);
+// S <- keep S + write k v^T, out = S^T q over each sequence's rows, S = state[slot][0 ...] [H, D, V] float32; with sums
+// [rows, H] (may be null) also n <- keep n + write k, sums = n . q, n = state[slot][sum_off ...] [H, D].  decay [H]: keep,
+// with write 1; or logs [rows, H, 2] of both.  q, k [.., H D], v [.., H V] float32 rows `stride` apart; act 1: through SiLU;
+// q times q_scale.  form 0: token by token; 1: the same for single tokens; 2: 64 tokens at a time on the tensor cores with
+// bfloat16 operands and float32 state, exponents and sums.
+int citlali_linear_memory(const float* q, const float* k, const float* v, size_t stride, int act, float q_scale,
+                          const float* decay, const float* logs, float* state, size_t state_stride, size_t sum_off,
+                          const int32_t* seq_start, const int32_t* seq_slot, int sequences, int H, int D, int V, float* out,
+                          float* sums, int form, cudaStream_t stream);
+// y = o (with sums: / (max(|sums|, floors) + 1e-6) a head), divided by the root mean square of each of `groups` equal parts
+// of a row (eps inside the root), times weight [H V], times sigmoid(gate[r * gate_stride + c]).
+int citlali_linear_memory_output(const float* o, const float* sums, const float* floors, const float* gate, size_t gate_stride,
+                                 const float* weight, void* y, int y_dtype, int rows, int H, int V, int groups, float eps,
+                                 cudaStream_t stream);
+
 // ---- attention over a window that keeps the first tokens ------------------------------------------------------------
 // proj [rows, proj_stride] float32 = q (nq d) | k (nkv d) | v (nkv vd).  Every channel passes a causal convolution (taps_w
 // [C, taps], no bias; kept inputs as in citlali_causal_conv; the caller stores them afterwards with citlali_conv_keep); q and
@@ -319,29 +349,42 @@ int citlali_attention_window(const void* q, int q_dtype, const void* k_pool, con
                              const int32_t* page_table, int table_stride, const int32_t* row_slot, const int32_t* row_pos,
                              void* out, int rows, int nq, int nkv, int d, int vd, int page_size, int window, int keep_first,
                              int max_keys, float scale, float softcap, const float* gate, size_t gate_stride,
-                             const float* sink, const float* turns, int turn_pairs, cudaStream_t stream);
+                             const float* sink, const float* turns, int turn_pairs, float* out32, cudaStream_t stream);
 // (sink, turns, turn_pairs: as citlali_attention_prefill takes them)
 
 // What attention without a convolution reads, from proj [rows, proj_stride] = q (nq d) | k (nkv d) | v (nkv vd) | ...: bias
 // (may be null), an RMS norm over all of q and over all of k with weights of those sizes (may both be null), the rotation of
 // the first rot_dims elements of a head (halves, or with rot_pairs neighbours) with cos and sin times amplitude, and with
 // v_freq [vd / 2] that of the whole value head (halves, or neighbours with v_pairs), whose cos and sin also go to turns
-// [rows, vd / 2].  q to q_out [rows, nq d], k and v to the row's place in the pools.
+// [rows, vd / 2].  q to q_out [rows, nq d], k and v to the row's place in the pools.  maps > 1: a head of d elements is `maps`
+// equal parts that score on their own; each part is rotated by itself (rot_dims of its elements) and q_out is [rows, nq maps
+// d]: query head h maps + s holds part s at its place in a row of d whose other parts are zeros.
 int citlali_heads_prepare(const float* proj, int proj_stride, const float* bias, const float* q_gain, const float* k_gain,
                           float eps, const float* inv_freq, int rot_dims, int rot_pairs, float amplitude, const float* v_freq,
                           int v_pairs, float* turns, const int32_t* row_slot, const int32_t* row_pos, const int32_t* page_table,
                           int table_stride, void* k_pool, void* v_pool, int cache_dtype, int page_size, void* q_out, int q_dtype,
-                          int rows, int nq, int nkv, int d, int vd, cudaStream_t stream);
+                          int rows, int nq, int nkv, int d, int vd, int maps, cudaStream_t stream);
+// out[r, h, :] = (o / sqrt(mean(o^2) + eps)) factor sigmoid(gate[r gate_stride + h]) with o = a[r, 2h, :] - lambda a[r, 2h + 1, :],
+// a [rows, 2 H, V] float32; gate may be null (no factor).
+int citlali_differential_output(const float* a, float lambda, float factor, float eps, const float* gate, size_t gate_stride,
+                                void* out, int out_dtype, int rows, int H, int V, cudaStream_t stream);
 
 // ---- routed experts ----------------------------------------------------------------------------------------------------
 // weights [rows, E] = softmax(logits) at the `top` best experts among those of the `keep` best of `groups` equal groups of
 // neighbours (a group's score is its largest score; groups <= 1: no groups), 0 elsewhere; chosen [rows, top] (may be
 // null) their indices, best first.
 // The chosen experts' weights are multiplied by weight_scale.  score_kind 1: the scores are sigmoid(logits), each by itself;
-// 2: the logits choose, and the weights are the softmax over the chosen.  Rows of logits are `stride` apart; bias [E] (may be
+// 2: the logits choose, and the weights are the softmax over the chosen.  correction [E] (may be null) is added to the scores
+// for every choice, of groups and of experts, and not to the weights; group_best 2: a group's score is the sum of its two
+// largest scores; renormalise: the chosen weights are divided by their sum (+ 1e-20) ahead of weight_scale.  Rows of logits are `stride` apart; bias [E] (may be
 // null) is added to them.  extra [rows] (may be null) = sigmoid of the column behind the experts'.
 int citlali_moe_route(const float* logits, float* weights, int32_t* chosen, int rows, int E, int groups, int keep, int top,
-                      float weight_scale, int score_kind, int stride, const float* bias, float* extra, cudaStream_t stream);
+                      float weight_scale, int score_kind, int stride, const float* bias, float* extra, const float* correction,
+                      int group_best, int renormalise, cudaStream_t stream);
+// act[r, e, j] = weights[r, e] max(z[r, e, j], 0)^2 over z [rows, E ff + tail_ff] (a zero weight: zeros, z not read); the tail's
+// factor is tail_weights[r] (null: 1).
+int citlali_expert_relu_squared(const void* z, int z_dtype, const float* weights, void* act, int act_dtype, int rows, int E, int ff,
+                                int tail_ff, const float* tail_weights, cudaStream_t stream);
 // act [rows, E ff + tail_ff] from gate_up [rows, 2 (E ff + tail_ff)], whose columns are, expert after expert, gate and up
 // alternating in runs of `run` (the last expert, which every row uses with weight 1, in runs of `tail_run`).  kind 0:
 // silu(g) u; kind 1: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).  Routed expert e's

@@ -234,6 +234,8 @@ struct DecodeOptions {
     const float* gate = nullptr;
     size_t gate_stride = 0;
     int turn_pairs = 0, dk = 0, dv = 0;
+    float* out32 = nullptr;            // the result in float32, rows out32_stride apart, instead of the rounded one
+    size_t out32_stride = 0;
 };
 
 __device__ __forceinline__ float sink_share(const DecodeOptions& opt, int head, float M) {      // M in units of log2
@@ -245,7 +247,8 @@ template <typename Value>
 __device__ __forceinline__ void store_head(const DecodeOptions& opt, int row, int head, int dv, __nv_bfloat16* out_head, int tid, Value value) {
     auto store = [&](int i, float r) {
         if (opt.gate) r *= 1.0f / (1.0f + expf(-opt.gate[(size_t)row * opt.gate_stride + (size_t)head * dv + i]));
-        out_head[i] = __float2bfloat16_rn(r);
+        if (opt.out32) opt.out32[(size_t)row * opt.out32_stride + (size_t)head * dv + i] = r;
+        else out_head[i] = __float2bfloat16_rn(r);
     };
     if (opt.turns) {
         const int half = dv / 2;
@@ -887,7 +890,7 @@ extern "C" int citlali_attention_decode_with(const void* q, int q_stride, const 
                                              size_t partial_floats, int32_t* counters, size_t counter_ints, int rows, int nq,
                                              int nkv, int head_dim, int value_dim, int page_size, int window, float scale,
                                              float softcap, const float* gate, size_t gate_stride, const float* sink,
-                                             const float* turns, int turn_pairs, cudaStream_t stream) {
+                                             const float* turns, int turn_pairs, float* out32, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || rows > 65535 || nq > 65535) {
         set_last_error("attention_decode_with: %d query heads over %d key/value heads, %d rows", nq, nkv, rows);
@@ -910,6 +913,8 @@ extern "C" int citlali_attention_decode_with(const void* q, int q_stride, const 
     opt.gate = gate;
     opt.gate_stride = gate_stride;
     opt.turn_pairs = turn_pairs;
+    opt.out32 = out32;
+    opt.out32_stride = (size_t)out_stride;
     opt.dk = head_dim;
     opt.dv = value_dim;
 #define CITLALI_TC(DD, EX) return launch_tc<DD, EX>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, \

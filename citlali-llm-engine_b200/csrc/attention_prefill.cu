@@ -45,7 +45,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                          __nv_bfloat16* __restrict__ out, int out_stride,
                          int nq, int nkv, int window, int keep_first, float scale_log2, float cap_in, float cap_out,
                          const float* __restrict__ gate, size_t gate_stride, const float* __restrict__ sink,
-                         const float2* __restrict__ turns, int turn_pairs, int dk_arg, int dv_arg) {
+                         const float2* __restrict__ turns, int turn_pairs, int dk_arg, int dv_arg, float* __restrict__ out32) {
     const int dk = EXACT ? D : dk_arg, dv = EXACT ? D : dv_arg;
     constexpr int kRowBytes = D * 2 + 16;
     constexpr int kTileBytes = kTileK * kRowBytes;
@@ -280,6 +280,11 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                 b0 *= 1.0f / (1.0f + expf(-g.x)); b1 *= 1.0f / (1.0f + expf(-g.y));
             }
         }
+        if (out32) {                                         // for a caller that goes on in float32
+            if (r0 < n_new) *reinterpret_cast<float2*>(out32 + (size_t)(row0 + r0) * out_stride + c) = make_float2(a0, a1);
+            if (r1 < n_new) *reinterpret_cast<float2*>(out32 + (size_t)(row0 + r1) * out_stride + c) = make_float2(b0, b1);
+            continue;
+        }
         if (r0 < n_new) *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + r0) * out_stride + c) = pack_bf16(a0, a1);
         if (r1 < n_new) *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + r1) * out_stride + c) = pack_bf16(b0, b1);
     }
@@ -290,7 +295,7 @@ static int launch(const void* q, int q_stride, const void* k_pool, const void* v
                   int page_table_stride, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_past,
                   void* out, int out_stride, int sequences, int max_new, int nq, int nkv, int window, int keep_first,
                   float scale, float softcap, const float* gate, size_t gate_stride, const float* sink, const float2* turns,
-                  int turn_pairs, int dk, int dv, cudaStream_t stream) {
+                  int turn_pairs, int dk, int dv, float* out32, cudaStream_t stream) {
     constexpr int smem = 5 * kTileK * (D * 2 + 16);
     auto kernel = attention_prefill_kernel<D, EXACT>;
     static bool configured = false;
@@ -307,7 +312,7 @@ static int launch(const void* q, int q_stride, const void* k_pool, const void* v
                                                  softcap > 0.0f ? 1.0f : scale * 1.4426950408889634f,
                                                  softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f,
                                                  softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f, gate, gate_stride, sink, turns,
-                                                 turn_pairs, dk, dv);
+                                                 turn_pairs, dk, dv, out32);
     return CITLALI_LAUNCH_CHECK();
 }
 
@@ -342,7 +347,7 @@ extern "C" int citlali_attention_prefill(const void* q, int q_stride, const void
                                          void* out, int out_stride, int sequences, int max_new,
                                          int nq, int nkv, int head_dim, int value_dim, int page_size, int window, int keep_first,
                                          float scale, float softcap, const float* gate, size_t gate_stride, const float* sink,
-                                         const float* turns, int turn_pairs, cudaStream_t stream) {
+                                         const float* turns, int turn_pairs, float* out32, cudaStream_t stream) {
     if (sequences <= 0 || max_new <= 0) return 0;
     if (!citlali_attention_prefill_supports_sizes(head_dim, value_dim, page_size)) {
         set_last_error("attention_prefill: no kernel for keys of %d and values of %d with pages of %d (multiples of 8 up to 256, "
@@ -357,13 +362,17 @@ extern "C" int citlali_attention_prefill(const void* q, int q_stride, const void
         set_last_error("attention_prefill: the gate's rows must be 8-byte aligned (row pitch %zu floats)", gate_stride);
         return kBadAlignment;
     }
-    if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 3u) || ((uintptr_t)turns & 15u)) {
+    if (out32 != nullptr && turns != nullptr) {
+        set_last_error("attention_prefill: an output that is turned back is not left in float32");
+        return kBadShape;
+    }
+    if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 3u) || ((uintptr_t)turns & 15u) || ((uintptr_t)out32 & 7u)) {
         set_last_error("attention_prefill: query rows must be 16-byte aligned (row pitch %d elements)", q_stride);
         return kBadAlignment;
     }
 #define CITLALI_FA(DD, EX) return fa::launch<DD, EX>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, seq_start, \
                                                       seq_slot, seq_past, out, out_stride, sequences, max_new, nq, nkv, window, keep_first, scale, \
-                                                      softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, head_dim, value_dim, stream)
+                                                      softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, head_dim, value_dim, out32, stream)
     if (head_dim == value_dim) {
         switch (head_dim) {
             case 16: CITLALI_FA(16, true);

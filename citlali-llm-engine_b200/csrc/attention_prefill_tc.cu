@@ -231,6 +231,7 @@ struct Params {
     const float* sink; const float2* turns; const float* gate;
     size_t gate_stride;
     int turn_pairs;
+    float* out32;                        // the result in float32 instead of the rounded one (rows out_stride apart)
 };
 
 // One of the block's two query tiles: its head, its first row within the sequence's new tokens, and the
@@ -667,6 +668,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         }
                     }
                 }
+                if constexpr (kWith) {
+                    if (p.out32) {
+                        if (store) {
+                            float* wide = p.out32 + (size_t)(row0 + me.q0 + r) * p.out_stride + (size_t)me.head * kD + half * kHalfKeys + c0;
+#pragma unroll
+                            for (int c = 0; c < 16; c += 4)
+                                *reinterpret_cast<float4*>(wide + c) = make_float4(__uint_as_float(ov[c]) * inv, __uint_as_float(ov[c + 1]) * inv,
+                                                                                  __uint_as_float(ov[c + 2]) * inv, __uint_as_float(ov[c + 3]) * inv);
+                        }
+                        continue;
+                    }
+                }
                 if (store) {
 #pragma unroll
                     for (int c = 0; c < 16; c += 8) {
@@ -711,7 +724,7 @@ static int launch_prefill_tc(const void* q, int q_stride, int total_rows, const 
                              const int32_t* seq_past, void* out, int out_stride, int sequences, int max_new, int nq, int nkv,
                              int head_dim, int page_size, int window, float scale, int32_t* error_flag, bool with, float softcap,
                              const float* gate, size_t gate_stride, const float* sink, const float* turns, int turn_pairs,
-                             cudaStream_t stream) {
+                             float* out32, cudaStream_t stream) {
     if (sequences <= 0 || max_new <= 0) return 0;
     if (!citlali_attention_prefill_tc_supports(head_dim, page_size)) {
         set_last_error("attention_prefill_tc: head size %d with pages of %d is not taken (128 and 64 only)", head_dim, page_size);
@@ -722,7 +735,7 @@ static int launch_prefill_tc(const void* q, int q_stride, int total_rows, const 
         return kBadShape;
     }
     if (q_stride % 8 != 0 || out_stride % 8 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)out & 15u) ||
-        ((uintptr_t)k_pool & 15u) || ((uintptr_t)v_pool & 15u) || ((uintptr_t)turns & 15u) || ((uintptr_t)gate & 15u) || (gate && gate_stride % 4 != 0)) {
+        ((uintptr_t)k_pool & 15u) || ((uintptr_t)v_pool & 15u) || ((uintptr_t)turns & 15u) || ((uintptr_t)gate & 15u) || ((uintptr_t)out32 & 15u) || (gate && gate_stride % 4 != 0)) {
         set_last_error("attention_prefill_tc: rows of q and out must be 16-byte aligned");
         return kBadAlignment;
     }
@@ -745,7 +758,7 @@ static int launch_prefill_tc(const void* q, int q_stride, int total_rows, const 
     p.cap_in = softcap > 0.0f ? 2.0f * log2e * scale / softcap : 0.0f;
     p.cap_out = softcap > 0.0f ? softcap * log2e : 0.0f;
     p.fixed_reference = p.cap_out > 0.0f && p.cap_out <= 100.0f ? 1 : 0;
-    p.sink = sink; p.turns = (const float2*)turns; p.gate = gate; p.gate_stride = gate_stride; p.turn_pairs = turn_pairs;
+    p.sink = sink; p.turns = (const float2*)turns; p.gate = gate; p.gate_stride = gate_stride; p.turn_pairs = turn_pairs; p.out32 = out32;
     const size_t smem = (size_t)6 * fatc::kTileBytes + 1024;
     auto kernel = with ? fatc::attention_prefill_tc_kernel<true> : fatc::attention_prefill_tc_kernel<false>;
     static bool configured[2] = {false, false};
@@ -771,7 +784,7 @@ extern "C" int citlali_attention_prefill_tc(const void* q, int q_stride, int tot
                                             int32_t* error_flag, cudaStream_t stream) {
     return launch_prefill_tc(q, q_stride, total_rows, k_pool, v_pool, pool_pages, page_table, page_table_stride, seq_start, seq_slot,
                              seq_past, out, out_stride, sequences, max_new, nq, nkv, head_dim, page_size, window, scale, error_flag,
-                             false, 0.0f, nullptr, 0, nullptr, nullptr, 0, stream);
+                             false, 0.0f, nullptr, 0, nullptr, nullptr, 0, nullptr, stream);
 }
 
 extern "C" int citlali_attention_prefill_tc_with(const void* q, int q_stride, int total_rows, const void* k_pool, const void* v_pool,
@@ -780,8 +793,8 @@ extern "C" int citlali_attention_prefill_tc_with(const void* q, int q_stride, in
                                                  int out_stride, int sequences, int max_new, int nq, int nkv, int head_dim,
                                                  int page_size, int window, float scale, int32_t* error_flag, float softcap,
                                                  const float* gate, size_t gate_stride, const float* sink, const float* turns,
-                                                 int turn_pairs, cudaStream_t stream) {
+                                                 int turn_pairs, float* out32, cudaStream_t stream) {
     return launch_prefill_tc(q, q_stride, total_rows, k_pool, v_pool, pool_pages, page_table, page_table_stride, seq_start, seq_slot,
                              seq_past, out, out_stride, sequences, max_new, nq, nkv, head_dim, page_size, window, scale, error_flag,
-                             true, softcap, gate, gate_stride, sink, turns, turn_pairs, stream);
+                             true, softcap, gate, gate_stride, sink, turns, turn_pairs, out32, stream);
 }

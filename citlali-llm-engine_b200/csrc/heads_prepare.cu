@@ -10,6 +10,10 @@
 // With v_freq the row's cosines and sines go to turns [rows, vd / 2] (cos, sin), from which the attention kernels turn their
 // output back.  Everything is float32 until the one rounding at the store.
 //
+// With maps > 1 a head of d elements is `maps` equal parts that score on their own (the maps of differential attention): each
+// part is rotated by itself, and a query head becomes `maps` heads of d whose other parts are zeros, so that one key of d
+// elements serves them all.
+//
 // One block a row, its size given by the projections' width alone (so are the orders of the sums).
 #include "api.h"
 #include "common.cuh"
@@ -44,7 +48,7 @@ struct HeadsArgs {
     const float *bias, *q_gain, *k_gain, *inv_freq, *v_freq;
     const int32_t *row_slot, *row_pos, *page_table;
     float2* turns;
-    int rot_dims, rot_pairs, v_pairs, table_stride, page_size, nq, nkv, d, vd;
+    int rot_dims, rot_pairs, v_pairs, table_stride, page_size, nq, nkv, d, vd, maps;
     float amplitude, eps;
 };
 
@@ -66,7 +70,7 @@ heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool
         trig[i] = is_v ? make_float2(cs, sn) : make_float2(cs * a.amplitude, sn * a.amplitude);
     }
     const float* x = a.proj + (size_t)row * a.proj_stride;
-    const int Cq = a.nq * a.d, Ck = a.nkv * a.d, Cv = a.nkv * a.vd;
+    const int Cq = a.nq * a.d, Ck = a.nkv * a.d, Cv = a.nkv * a.vd, dm = a.d / a.maps;
     float q_inv = 1.0f, k_inv = 1.0f;
     if (a.q_gain) {
         float sq = 0.0f, sk = 0.0f;
@@ -116,7 +120,7 @@ heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool
         const bool is_q = c < Cq, is_v = c >= Cq + Ck;
         const int at = is_q ? c : (is_v ? c - Cq - Ck : c - Cq);
         const int n = is_v ? a.vd : a.d;
-        const int head = at / n, i = at % n;
+        const int head = at / n, in_head = at % n, i = is_v || a.maps == 1 ? in_head : in_head % dm;
         const int h = is_v ? vhalf : half;                    // pairs of the rotation
         const bool pairs = is_v ? a.v_pairs != 0 : a.rot_pairs != 0;
         const float2* t = is_v ? trig + half : trig;
@@ -149,9 +153,16 @@ heads_prepare_kernel(HeadsArgs a, T* __restrict__ k_pool, T* __restrict__ v_pool
                 }
             }
         }
-        if (is_q) put<TQ, N>(q_out + (size_t)row * Cq + c, v);
+        if (is_q && a.maps > 1) {
+            TQ* dst = q_out + ((size_t)row * Cq + (size_t)head * a.d) * a.maps + in_head;
+            const float zeros[N] = {};
+            for (int s = 0; s < a.maps; ++s)
+                if (s == in_head / dm) put<TQ, N>(dst + (size_t)s * a.d, v);
+                else put<TQ, N>(dst + (size_t)s * a.d, zeros);
+        }
+        else if (is_q) put<TQ, N>(q_out + (size_t)row * Cq + c, v);
         else if (is_v) put<T, N>(v_pool + (cache_row + (size_t)head * a.page_size) * a.vd + i, v);
-        else put<T, N>(k_pool + (cache_row + (size_t)head * a.page_size) * a.d + i, v);
+        else put<T, N>(k_pool + (cache_row + (size_t)head * a.page_size) * a.d + in_head, v);
     }
 }
 
@@ -165,13 +176,17 @@ extern "C" int citlali_heads_prepare(const float* proj, int proj_stride, const f
                                      const float* v_freq, int v_pairs, float* turns, const int32_t* row_slot,
                                      const int32_t* row_pos, const int32_t* page_table, int table_stride, void* k_pool,
                                      void* v_pool, int cache_dtype, int page_size, void* q_out, int q_dtype, int rows, int nq,
-                                     int nkv, int d, int vd, cudaStream_t stream) {
+                                     int nkv, int d, int vd, int maps, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || vd <= 0 || page_size <= 0 || (q_gain == nullptr) != (k_gain == nullptr)) {
         set_last_error("heads_prepare: %d query heads over %d key/value heads of %d (values %d)", nq, nkv, d, vd);
         return kBadShape;
     }
-    if (rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > d || (rot_dims > 0 && inv_freq == nullptr) ||
+    if (maps < 1 || d % maps != 0) {
+        set_last_error("heads_prepare: heads of %d do not split into %d equal parts", d, maps);
+        return kBadShape;
+    }
+    if (rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > d / maps || (rot_dims > 0 && inv_freq == nullptr) ||
         (v_freq != nullptr && (vd % 2 != 0 || turns == nullptr))) {
         set_last_error("heads_prepare: %d rotated elements must be even and at most the head size %d; rotated values (%d) need an "
                        "even size and room for their cosines", rot_dims, d, vd);
@@ -183,9 +198,9 @@ extern "C" int citlali_heads_prepare(const float* proj, int proj_stride, const f
         return kTooLarge;
     }
     HeadsArgs a{proj, (size_t)proj_stride, bias, q_gain, k_gain, inv_freq, v_freq, row_slot, row_pos, page_table, (float2*)turns,
-                rot_dims, rot_pairs, v_pairs, table_stride, page_size, nq, nkv, d, vd, amplitude, eps};
+                rot_dims, rot_pairs, v_pairs, table_stride, page_size, nq, nkv, d, vd, maps, amplitude, eps};
     // four elements at a time: no piece crosses a head, a rotation's half or its end
-    const bool vec = d % 4 == 0 && vd % 4 == 0 && proj_stride % 4 == 0 && rot_dims % 4 == 0 && (rot_pairs || rot_dims % 8 == 0) &&
+    const bool vec = (d / maps) % 4 == 0 && vd % 4 == 0 && proj_stride % 4 == 0 && rot_dims % 4 == 0 && (rot_pairs || rot_dims % 8 == 0) &&
                      (v_freq == nullptr || v_pairs || vd % 8 == 0) &&
                      (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)k_pool |
                        (uintptr_t)v_pool | (uintptr_t)q_out) & 15u) == 0;

@@ -8,7 +8,10 @@
 //                   chosen (of equal scores the lower index first); their weights are the scores themselves, not
 //                   renormalised (score_kind 0 and 1).  weights [rows, E] receives the score of a chosen expert and 0 for every other; chosen
 //                   [rows, top] the indices, best first.  With `extra` the column behind the experts' logits is one more number
-//                   of the row (an expert that every row uses), and extra [rows] receives its sigmoid.
+//                   of the row (an expert that every row uses), and extra [rows] receives its sigmoid.  With `correction` a
+//                   number an expert is added to the scores wherever groups and experts are compared (choice scores, which
+//                   may be negative); weights are made of the scores without it.  group_best 2: a group's score is the sum
+//                   of its two largest choice scores.  renormalise: the chosen weights are divided by their sum (+ 1e-20).
 //   moe_scale       act[r, e, j] *= weights[r, e] over act [rows, E, ff]: after this, one product with every expert's output
 //                   matrix side by side is the weighted sum of the chosen experts' outputs (the others contribute zeros).
 #include "api.h"
@@ -23,7 +26,7 @@ template <int PER>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, int32_t* __restrict__ chosen, int rows, int E,
                  int groups, int keep, int top, float weight_scale, int score_kind, int stride, const float* __restrict__ bias,
-                 float* __restrict__ extra) {
+                 float* __restrict__ extra, const float* __restrict__ correction, int group_best, int renormalise) {
     dependents_may_launch();
     wait_for_predecessor();
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -54,6 +57,12 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
 #pragma unroll
         for (int j = 0; j < PER; ++j) s[j] = s[j] / sum;
     }
+    float choice[PER];                                       // what groups and experts are compared by
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int e = lane + 32 * j;
+        choice[j] = correction && e < E ? s[j] + correction[e] : s[j];
+    }
     // which experts may be chosen: bit j of `open` for expert lane + 32 j
     unsigned open = 0;
 #pragma unroll
@@ -62,18 +71,31 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
     if (groups > 1 && keep < groups) {
         const int per = E / groups;
         unsigned kept_mine = 0;                              // groups are looked at one after another; `keep` rounds
-        // a group's score: the largest score in it.  Lane l keeps the scores of groups l, l + 32, ... (at most 16 each).
+        // a group's score: the largest score in it, or the sum of its two largest.  Lane l keeps the scores of groups l, l + 32, ... (at most 16 each).
         float gs[PER];
 #pragma unroll
         for (int j = 0; j < PER; ++j) gs[j] = -INFINITY;
         for (int grp = 0; grp < groups; ++grp) {
-            float best = -INFINITY;
+            float best = -INFINITY, second = -INFINITY;
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const int e = lane + 32 * j;
-                if (e < E && e / per == grp) best = fmaxf(best, s[j]);
+                if (e < E && e / per == grp) {
+                    second = fmaxf(second, fminf(best, choice[j]));
+                    best = fmaxf(best, choice[j]);
+                }
             }
-            best = warp_max(best);
+            if (group_best == 2) {
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, second, o);
+                    second = fmaxf(fminf(best, ob), fmaxf(second, os));
+                    best = fmaxf(best, ob);
+                }
+                if (per > 1) best += second;
+            } else {
+                best = warp_max(best);
+            }
 #pragma unroll
             for (int j = 0; j < PER; ++j)
                 if (grp == lane + 32 * j) gs[j] = best;
@@ -114,7 +136,7 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
             const int e = lane + 32 * j;
-            if ((open >> j & 1u) && !(taken >> j & 1u) && (s[j] > best || (s[j] == best && e < arg))) { best = s[j]; arg = e; }
+            if ((open >> j & 1u) && !(taken >> j & 1u) && (choice[j] > best || (choice[j] == best && e < arg))) { best = choice[j]; arg = e; }
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -141,6 +163,15 @@ moe_route_kernel(const float* __restrict__ logits, float* __restrict__ weights, 
         sum = warp_sum(sum);
 #pragma unroll
         for (int j = 0; j < PER; ++j) s[j] = s[j] / sum;
+    }
+    if (renormalise) {
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < PER; ++j)
+            if (taken >> j & 1u) sum += s[j];
+        sum = warp_sum(sum) + 1e-20f;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) s[j] /= sum;
     }
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
@@ -191,10 +222,14 @@ using namespace citlali;
 
 extern "C" int citlali_moe_route(const float* logits, float* weights, int32_t* chosen, int rows, int E, int groups, int keep,
                                  int top, float weight_scale, int score_kind, int stride, const float* bias, float* extra,
-                                 cudaStream_t stream) {
+                                 const float* correction, int group_best, int renormalise, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (score_kind < 0 || score_kind > 2) {
         set_last_error("moe_route: score kind %d is neither softmax (0), sigmoid (1) nor a softmax over the chosen (2)", score_kind);
+        return kBadShape;
+    }
+    if (group_best != 1 && group_best != 2) {
+        set_last_error("moe_route: a group's score is its largest (1) or its two largest scores (2), not %d", group_best);
         return kBadShape;
     }
     if (stride < E + (extra ? 1 : 0)) {
@@ -211,7 +246,7 @@ extern "C" int citlali_moe_route(const float* logits, float* weights, int32_t* c
     }
     auto go = [&](auto kernel) {
         launch_kernel(kernel, (rows + 3) / 4, 128, 0, stream, logits, weights, chosen, rows, E, groups, keep, top, weight_scale, score_kind,
-                      stride, bias, extra);
+                      stride, bias, extra, correction, group_best, renormalise);
     };
     if (E <= 32) go(moe_route_kernel<1>);
     else if (E <= 64) go(moe_route_kernel<2>);

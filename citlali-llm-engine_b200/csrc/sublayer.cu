@@ -6,6 +6,9 @@
 //   layer_norm_rows  out[i] = layer_norm(x[index[i]]) * w, rounded once (the model's last norm).
 //   cast_rows        float32 -> the compute dtype.
 //   scaled_sum       out = a * l + b * r (two mixers side by side).
+//   normed_pair_sum  the same of the two after an RMS norm of each with a weight of its own.
+//   add_rows_norm    x[r] += x0[r] + step (ahead of a pass over layers that repeat) and the norm in front of the next
+//                    sub-layer.
 // One block a row; the row waits in shared memory between the passes (mean, then deviations, then the store), so every
 // row is read from global memory once.
 #include "api.h"
@@ -314,6 +317,122 @@ layer_norm_chain_vec_kernel(const float* __restrict__ y, const float* __restrict
     }
 }
 
+// x[r] += x0[r] (x0 may be null) + step, and with a gain out[r] = layer_norm(x[r]) * gain + bias.  One block a row; a thread
+// keeps NV runs of W neighbouring elements in registers (W 4: rows of a multiple of four, 16-byte words; a row is at most
+// NV W threads).  The order of the sums follows the row's length alone.
+template <int W>
+__device__ __forceinline__ void load_run(const float* p, float (&v)[W]) {
+    if constexpr (W == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+        v[0] = p[0];
+    }
+}
+template <int W, typename T>
+__device__ __forceinline__ void store_run(T* p, const float (&v)[W]) {
+    if constexpr (W == 4) store4(p, (size_t)0, make_float4(v[0], v[1], v[2], v[3]));
+    else stf(p, 0, v[0]);
+}
+
+template <typename TO, int W, int NV>
+__global__ void __launch_bounds__(1024)
+add_rows_norm_kernel(float* __restrict__ x, const float* __restrict__ x0, const float* __restrict__ step,
+                     const float* __restrict__ gain, const float* __restrict__ bias, TO* __restrict__ out, int hidden, float eps) {
+    __shared__ float scratch[32];
+    dependents_may_launch();
+    wait_for_predecessor();
+    const size_t base = (size_t)blockIdx.x * hidden;
+    float v[NV][W];
+    float s = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * W;
+#pragma unroll
+        for (int e = 0; e < W; ++e) v[c][e] = 0.0f;
+        if (i < hidden) {
+            float t[W];
+            load_run<W>(x + base + i, v[c]);
+            if (x0) {
+                load_run<W>(x0 + base + i, t);
+#pragma unroll
+                for (int e = 0; e < W; ++e) v[c][e] += t[e];
+            }
+            load_run<W>(step + i, t);
+#pragma unroll
+            for (int e = 0; e < W; ++e) { v[c][e] += t[e]; s += v[c][e]; }
+            store_run<W>(x + base + i, v[c]);
+        }
+    }
+    if (gain == nullptr) return;
+    const float mean = block_sum(s, scratch) / (float)hidden;
+    float ss = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c)
+        if ((c * blockDim.x + threadIdx.x) * W < hidden) {
+#pragma unroll
+            for (int e = 0; e < W; ++e) { v[c][e] -= mean; ss = fmaf(v[c][e], v[c][e], ss); }
+        }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * W;
+        if (i < hidden) {
+            float g[W], b[W];
+            load_run<W>(gain + i, g);
+#pragma unroll
+            for (int e = 0; e < W; ++e) b[e] = 0.0f;
+            if (bias) load_run<W>(bias + i, b);
+#pragma unroll
+            for (int e = 0; e < W; ++e) v[c][e] = v[c][e] * inv * g[e] + b[e];
+            store_run<W>(out + base + i, v[c]);
+        }
+    }
+}
+
+// out[r] = a rms(l[r]) wl + b rms(r[r]) wr.
+template <int W, int NV>
+__global__ void __launch_bounds__(1024)
+normed_pair_sum_kernel(float a, const float* l, const float* __restrict__ wl, float b, const float* r, const float* __restrict__ wr,
+                       float* out, int hidden, float eps_l, float eps_r) {
+    __shared__ float scratch[32];
+    dependents_may_launch();
+    wait_for_predecessor();
+    const size_t base = (size_t)blockIdx.x * hidden;
+    float x[NV][W], y[NV][W];
+    float sl = 0.0f, sr = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * W;
+        if (i < hidden) {
+            load_run<W>(l + base + i, x[c]);
+            load_run<W>(r + base + i, y[c]);
+#pragma unroll
+            for (int e = 0; e < W; ++e) { sl = fmaf(x[c][e], x[c][e], sl); sr = fmaf(y[c][e], y[c][e], sr); }
+        }
+    }
+    const float fl = a / sqrtf(block_sum(sl, scratch) / (float)hidden + eps_l);
+    const float fr = b / sqrtf(block_sum(sr, scratch) / (float)hidden + eps_r);
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * W;
+        if (i < hidden) {
+            float g[W], h[W];
+            load_run<W>(wl + i, g);
+            load_run<W>(wr + i, h);
+#pragma unroll
+            for (int e = 0; e < W; ++e) x[c][e] = x[c][e] * fl * g[e] + y[c][e] * fr * h[e];
+            store_run<W>(out + base + i, x[c]);
+        }
+    }
+}
+
+// threads a row of `hidden` elements in runs of W: by the row's length alone
+static int run_threads(int hidden, int W) {
+    const int t = ((hidden / W + 31) / 32) * 32;
+    return t < 64 ? 64 : (t > 1024 ? 1024 : t);
+}
+
 static int grid_for(size_t n) {
     const size_t blocks = (n + 255) / 256;
     return (int)(blocks < 8192 ? (blocks ? blocks : 1) : 8192);
@@ -428,4 +547,48 @@ extern "C" int citlali_layer_norm_chain(const float* y, const float* in_bias, co
         launch_kernel(kernel, rows, threads, smem, stream, y, in_bias, g1, b1, x, (TE*)emit, g2, b2, (TE*)out2, hidden, eps1, eps2);
         return CITLALI_LAUNCH_CHECK();
     });
+}
+
+extern "C" int citlali_add_rows_norm(float* x, const float* x0, const float* step, const float* gain, const float* bias, void* out,
+                                     int out_dtype, int rows, int hidden, float eps, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (hidden <= 0 || hidden > 16384 || step == nullptr || (gain != nullptr && out == nullptr)) {
+        set_last_error("add_rows_norm: rows of %d elements (at most 16,384); a norm needs an output", hidden);
+        return kBadShape;
+    }
+    const uintptr_t together = (uintptr_t)x | (uintptr_t)x0 | (uintptr_t)step | (uintptr_t)gain | (uintptr_t)bias | (uintptr_t)out;
+    return CITLALI_DISPATCH_FLOAT(out_dtype, TO, [&] {
+        auto go = [&](auto kernel, int W) {
+            launch_kernel(kernel, rows, run_threads(hidden, W), 0, stream, x, x0, step, gain, bias, (TO*)out, hidden, eps);
+        };
+        if (hidden % 4 == 0 && (together & 15u) == 0) {
+            if (hidden <= 4096) go(add_rows_norm_kernel<TO, 4, 1>, 4);
+            else if (hidden <= 8192) go(add_rows_norm_kernel<TO, 4, 2>, 4);
+            else go(add_rows_norm_kernel<TO, 4, 4>, 4);
+        } else if (hidden <= 1024) go(add_rows_norm_kernel<TO, 1, 1>, 1);
+        else if (hidden <= 4096) go(add_rows_norm_kernel<TO, 1, 4>, 1);
+        else go(add_rows_norm_kernel<TO, 1, 16>, 1);
+        return CITLALI_LAUNCH_CHECK();
+    });
+}
+
+extern "C" int citlali_normed_pair_sum(float a, const float* l, const float* wl, float b, const float* r, const float* wr, float* out,
+                                       int rows, int hidden, float eps_l, float eps_r, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (hidden <= 0 || hidden > 16384) {
+        set_last_error("normed_pair_sum: rows of %d elements (at most 16,384)", hidden);
+        return kTooLarge;
+    }
+    const uintptr_t together = (uintptr_t)l | (uintptr_t)wl | (uintptr_t)r | (uintptr_t)wr | (uintptr_t)out;
+    auto go = [&](auto kernel, int W) {
+        launch_kernel(kernel, rows, run_threads(hidden, W), 0, stream, a, l, wl, b, r, wr, out, hidden, eps_l, eps_r);
+    };
+    if (hidden % 4 == 0 && (together & 15u) == 0) {
+        if (hidden <= 4096) go(normed_pair_sum_kernel<4, 1>, 4);
+        else if (hidden <= 8192) go(normed_pair_sum_kernel<4, 2>, 4);
+        else go(normed_pair_sum_kernel<4, 4>, 4);
+    } else if (hidden <= 1024) go(normed_pair_sum_kernel<1, 1>, 1);
+    else if (hidden <= 4096) go(normed_pair_sum_kernel<1, 4>, 1);
+    else go(normed_pair_sum_kernel<1, 16>, 1);
+    return CITLALI_LAUNCH_CHECK();
 }

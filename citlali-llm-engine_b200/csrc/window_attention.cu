@@ -10,7 +10,7 @@
 //   attention_window     one block a (row, query head): keys j <= pos with pos - j < window or j < keep_first (window 0:
 //                        every key); scores, softmax and the weighted sum in float32; with a soft cap c the scaled score s
 //                        becomes c tanh(s / c) before the softmax; with a gate the head's output element i is multiplied
-//                        by sigmoid(gate[row, head vd + i]).  With sinks the softmax's denominator also counts
+//                        by sigmoid(gate[row, head vd + i]); with out32 the result stays float32 (whatever q is).  With sinks the softmax's denominator also counts
 //                        exp(sink[head]), neither scaled nor capped.  With turns the head's output, whose values were rotated
 //                        before they were cached, is turned back by the row's own angles (ahead of the gate).  The keys are dealt to 32 groups of
 //                        eight lanes by their place among the visible keys, each group keeps a running softmax of its own,
@@ -145,7 +145,8 @@ attention_window_kernel(const TQ* __restrict__ q, const T* __restrict__ k_pool, 
                         const int32_t* __restrict__ page_table, int table_stride, const int32_t* __restrict__ row_slot,
                         const int32_t* __restrict__ row_pos, TQ* __restrict__ out, int nq, int nkv, int d, int vd,
                         int page_size, int window, int keep_first, float scale, float softcap, const float* __restrict__ gate,
-                        size_t gate_stride, const float* __restrict__ sink, const float2* __restrict__ turns, int turn_pairs) {
+                        size_t gate_stride, const float* __restrict__ sink, const float2* __restrict__ turns, int turn_pairs,
+                        float* __restrict__ out32) {
     extern __shared__ float smem[];                            // [32 groups][vd] weighted sums, then [32] maxima, [32] sums
     dependents_may_launch();
     wait_for_predecessor();
@@ -272,7 +273,8 @@ attention_window_kernel(const TQ* __restrict__ q, const T* __restrict__ k_pool, 
     };
     auto store = [&](int i, float r) {
         if (gate) r *= 1.0f / (1.0f + expf(-gate[(size_t)row * gate_stride + (size_t)head * vd + i]));
-        stf(out, (size_t)row * nq * vd + (size_t)head * vd + i, r);
+        if (out32) out32[(size_t)row * nq * vd + (size_t)head * vd + i] = r;
+        else stf(out, (size_t)row * nq * vd + (size_t)head * vd + i, r);
     };
     if (turns) {
         const int half = vd / 2;
@@ -292,12 +294,12 @@ template <typename T, typename TQ, int PL, bool VEC>
 static int launch_window(const void* q, const void* k_pool, const void* v_pool, const int32_t* page_table, int table_stride,
                          const int32_t* row_slot, const int32_t* row_pos, void* out, int rows, int nq, int nkv, int d, int vd,
                          int page_size, int window, int keep_first, float scale, float softcap, const float* gate,
-                         size_t gate_stride, const float* sink, const float2* turns, int turn_pairs, cudaStream_t stream) {
+                         size_t gate_stride, const float* sink, const float2* turns, int turn_pairs, float* out32, cudaStream_t stream) {
     const size_t smem = (size_t)(32 * vd + 64) * sizeof(float);
     dim3 grid(rows, nq);
     launch_kernel(attention_window_kernel<T, TQ, PL, VEC>, grid, kWinWarps * 32, smem, stream, (const TQ*)q, (const T*)k_pool,
                   (const T*)v_pool, page_table, table_stride, row_slot, row_pos, (TQ*)out, nq, nkv, d, vd, page_size, window,
-                  keep_first, scale, softcap, gate, gate_stride, sink, turns, turn_pairs);
+                  keep_first, scale, softcap, gate, gate_stride, sink, turns, turn_pairs, out32);
     return CITLALI_LAUNCH_CHECK();
 }
 
@@ -341,7 +343,7 @@ extern "C" int citlali_attention_window(const void* q, int q_dtype, const void* 
                                         const int32_t* row_pos, void* out, int rows, int nq, int nkv, int d, int vd,
                                         int page_size, int window, int keep_first, int max_keys, float scale,
                                         float softcap, const float* gate, size_t gate_stride, const float* sink,
-                                        const float* turns, int turn_pairs, cudaStream_t stream) {
+                                        const float* turns, int turn_pairs, float* out32, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (turns != nullptr && vd % 2 != 0) {
         set_last_error("attention_window: values of %d elements have no pairs to turn back", vd);
@@ -364,14 +366,14 @@ extern "C" int citlali_attention_window(const void* q, int q_dtype, const void* 
     do {                                                                                                                  \
         if (vec) {                                                                                                        \
             if constexpr (sizeof(T) == 2) {                                                                               \
-                if (big <= 64) return launch_window<T, TQ, 8, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
-                if (big <= 128) return launch_window<T, TQ, 16, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
-                return launch_window<T, TQ, 32, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
+                if (big <= 64) return launch_window<T, TQ, 8, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
+                if (big <= 128) return launch_window<T, TQ, 16, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
+                return launch_window<T, TQ, 32, true>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
             }                                                                                                             \
         }                                                                                                                 \
-        if (big <= 64) return launch_window<T, TQ, 8, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
-        if (big <= 128) return launch_window<T, TQ, 16, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
-        return launch_window<T, TQ, 32, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, stream); \
+        if (big <= 64) return launch_window<T, TQ, 8, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
+        if (big <= 128) return launch_window<T, TQ, 16, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
+        return launch_window<T, TQ, 32, false>(q, k_pool, v_pool, page_table, table_stride, row_slot, row_pos, out, rows, nq, nkv, d, vd, page_size, window, keep_first, scale, softcap, gate, gate_stride, sink, (const float2*)turns, turn_pairs, out32, stream); \
     } while (0)
     return CITLALI_DISPATCH_FLOAT(cache_dtype, T, [&] {
         return CITLALI_DISPATCH_FLOAT(q_dtype, TQ, [&]() -> int { CITLALI_WINDOW(T, TQ); });

@@ -326,8 +326,8 @@ def attention_prefill(q, q_stride, k_pool, v_pool, page_table, seq_start, seq_sl
     _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, sink, turns)
     vd = head_dim if value_dim is None else value_dim
     _check_sink_and_turns(sink, turns, nq, out.shape[0], vd)
-    require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
-            "attention_prefill: bfloat16 only")
+    require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype in _OUT_DTYPES,
+            "attention_prefill: bfloat16 only (the result may be left in float32)")
     require(gate is None or (gate.is_cuda and gate.dtype == torch.float32 and gate.stride(1) == 1
                              and gate.shape == (out.shape[0], nq * vd)), "attention_prefill: the gate does not fit")
     _check(lib().citlali_attention_prefill(
@@ -335,7 +335,10 @@ def attention_prefill(q, q_stride, k_pool, v_pool, page_table, seq_start, seq_sl
         _ptr(seq_start), _ptr(seq_slot), _ptr(seq_past), _ptr(out), _i(out.shape[1]), _i(sequences), _i(max_new),
         _i(nq), _i(nkv), _i(head_dim), _i(vd), _i(page_size), _i(window or 0), _i(keep_first or 0), _f(scale),
         _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink), _ptr(turns),
-        _i(1 if turn_pairs else 0), _stream()), "attention_prefill")
+        _i(1 if turn_pairs else 0), _ptr(out if out.dtype == torch.float32 else None), _stream()), "attention_prefill")
+
+
+_OUT_DTYPES = (torch.bfloat16, torch.float32)
 
 
 def _check_sink_and_turns(sink, turns, heads, rows, value_dim):
@@ -350,16 +353,17 @@ def attention_prefill_tc(q, q_stride, k_pool, v_pool, page_table, seq_start, seq
     """Prompt attention on tcgen05 (head size 128, pages of 64).  ``softcap``, ``gate``, ``sink``, ``turns``, ``turn_pairs``: see
     :func:`attention_prefill`."""
     _need_cuda(k_pool, v_pool, page_table, seq_start, seq_slot, seq_past, out, error_flag, sink, turns)
-    if softcap or gate is not None or sink is not None or turns is not None:
-        require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
-                "attention_prefill_tc: bfloat16 only")
+    if softcap or gate is not None or sink is not None or turns is not None or out.dtype == torch.float32:
+        require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype in _OUT_DTYPES,
+                "attention_prefill_tc: bfloat16 only (the result may be left in float32)")
         _check_sink_and_turns(sink, turns, nq, out.shape[0], head_dim)
         _check(lib().citlali_attention_prefill_tc_with(
             _ptr(q), _i(q_stride), _i(q.shape[0]), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(page_table),
             _i(page_table.shape[1]), _ptr(seq_start), _ptr(seq_slot), _ptr(seq_past), _ptr(out), _i(out.shape[1]),
             _i(sequences), _i(max_new), _i(nq), _i(nkv), _i(head_dim), _i(page_size), _i(window or 0), _f(scale),
             _ptr(error_flag), _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink),
-            _ptr(turns), _i(1 if turn_pairs else 0), _stream()), "attention_prefill_tc")
+            _ptr(turns), _i(1 if turn_pairs else 0), _ptr(out if out.dtype == torch.float32 else None), _stream()),
+            "attention_prefill_tc")
         return
     require(q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
             "attention_prefill_tc: bfloat16 only")
@@ -398,7 +402,7 @@ def attention_decode_with(q, kv, batch, out, nq, nkv, d, vd, window, scale, soft
     turned-back outputs (see :func:`attention_prefill`)."""
     _need_cuda(q, kv.keys, kv.values, kv.page_table, out, sink, turns)
     rows = out.shape[0]
-    require(q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    require(q.dtype == torch.bfloat16 and kv.keys.dtype == torch.bfloat16 and out.dtype in _OUT_DTYPES
             and q.shape == (rows, nq * d) and out.shape == (rows, nq * vd), "attention_decode_with: shapes or dtypes do not fit")
     _check_sink_and_turns(sink, turns, nq, rows, vd)
     l = lib()
@@ -412,7 +416,7 @@ def attention_decode_with(q, kv, batch, out, nq, nkv, d, vd, window, scale, soft
         _ptr(batch.row_slot), _ptr(batch.row_pos), _ptr(out), _i(out.shape[1]), _ptr(ws), _sz(ws.numel() // 4), _ptr(counters),
         _sz(counters.numel() // 4), _i(rows), _i(nq), _i(nkv), _i(d), _i(vd), _i(kv.page_size), _i(int(window or 0)), _f(scale),
         _f(float(softcap or 0.0)), _ptr(gate), _sz(gate.stride(0) if gate is not None else 0), _ptr(sink), _ptr(turns),
-        _i(1 if turn_pairs else 0), _stream()), "attention_decode_with")
+        _i(1 if turn_pairs else 0), _ptr(out if out.dtype == torch.float32 else None), _stream()), "attention_decode_with")
 
 
 _sm_count = {}
@@ -744,6 +748,28 @@ def cast_rows(x, out):
     _check(lib().citlali_cast_rows(_ptr(x), _ptr(out), _i(_dtype_code(out)), _sz(x.numel()), _stream()), "cast_rows")
 
 
+def add_rows_norm(x, x0, step, gain=None, bias=None, eps=0.0, out=None):
+    """``x += x0 + step`` (``x0`` None: only the vector); with ``gain`` also ``out = layer_norm(x) * gain + bias``."""
+    _need_cuda(x, x0, step, gain, bias, out)
+    rows, hidden = x.shape
+    require(x.dtype == torch.float32 and (x0 is None or (x0.dtype == torch.float32 and x0.shape == x.shape))
+            and all(v is None or (v.dtype == torch.float32 and v.numel() == hidden) for v in (step, gain, bias))
+            and (gain is None) == (out is None) and (out is None or out.shape == x.shape), "add_rows_norm: shapes or dtypes do not fit")
+    _check(lib().citlali_add_rows_norm(_ptr(x), _ptr(x0), _ptr(step), _ptr(gain), _ptr(bias), _ptr(out),
+                                       _i(_dtype_code(out) if out is not None else _F32), _i(rows), _i(hidden), _f(eps), _stream()),
+           "add_rows_norm")
+
+
+def normed_pair_sum(a, left, left_gain, left_eps, b, right, right_gain, right_eps, out):
+    """``out = a rms(left) left_gain + b rms(right) right_gain`` (float32; ``out`` may be one of the two)."""
+    _need_cuda(left, left_gain, right, right_gain, out)
+    rows, hidden = out.shape
+    require(all(t.dtype == torch.float32 for t in (left, left_gain, right, right_gain, out)) and left.shape == right.shape == out.shape
+            and left_gain.numel() == right_gain.numel() == hidden, "normed_pair_sum: float32 tensors of one shape and gains of a row's size")
+    _check(lib().citlali_normed_pair_sum(_f(a), _ptr(left), _ptr(left_gain), _f(b), _ptr(right), _ptr(right_gain), _ptr(out), _i(rows),
+                                         _i(hidden), _f(left_eps), _f(right_eps), _stream()), "normed_pair_sum")
+
+
 def scaled_sum(a, left, b, right, out):
     """``out = a * left + b * right`` (float32; ``out`` may be one of them)."""
     _need_cuda(left, right, out)
@@ -855,15 +881,16 @@ def conv_heads_prepare(proj, taps_w, state, conv_off, q_gain, k_gain, inv_freq, 
 
 
 def heads_prepare(proj, batch, kv, q_out, nq, nkv, d, vd, bias=None, q_gain=None, k_gain=None, eps=0.0, inv_freq=None,
-                  rot_dims=0, rot_pairs=False, amplitude=1.0, v_freq=None, v_pairs=False, turns=None):
+                  rot_dims=0, rot_pairs=False, amplitude=1.0, v_freq=None, v_pairs=False, turns=None, maps=1):
     """Bias, a norm over all of q and over all of k (``q_gain``/``k_gain`` of those sizes), rotations of q and k (``inv_freq``)
     and of v (``v_freq``; its cosines and sines go to ``turns`` [rows, vd / 2, 2]) and the cache write, in one pass over the
-    projection's rows.  ``proj`` may be wider than q | k | v."""
+    projection's rows.  ``proj`` may be wider than q | k | v.  ``maps`` > 1: heads of ``d`` elements are that many parts which score
+    on their own; ``q_out`` is [rows, nq maps d], a part at its place among zeros (see ``citlali_heads_prepare``)."""
     _need_cuda(proj, bias, q_gain, k_gain, inv_freq, v_freq, turns, kv.keys, kv.values, kv.page_table, q_out)
     rows = proj.shape[0]
     C = (nq + nkv) * d + nkv * vd
     f32 = lambda t, n: t is None or (t.dtype == torch.float32 and t.numel() == n)
-    require(proj.dtype == torch.float32 and proj.shape[1] >= C and q_out.shape == (rows, nq * d) and kv.keys.shape[-1] == d
+    require(proj.dtype == torch.float32 and proj.shape[1] >= C and q_out.shape == (rows, nq * maps * d) and kv.keys.shape[-1] == d
             and kv.values.shape[-1] == vd and kv.keys.shape[-3] == nkv and kv.keys.dtype == kv.values.dtype and f32(bias, C)
             and f32(q_gain, nq * d) and f32(k_gain, nkv * d) and (rot_dims == 0 or (inv_freq is not None and f32(inv_freq, rot_dims // 2)))
             and f32(v_freq, vd // 2) and (v_freq is None or (turns is not None and f32(turns, rows * vd))),
@@ -873,7 +900,20 @@ def heads_prepare(proj, batch, kv, q_out, nq, nkv, d, vd, bias=None, q_gain=None
         _i(1 if rot_pairs else 0), _f(amplitude), _ptr(v_freq), _i(1 if v_pairs else 0), _ptr(turns), _ptr(batch.row_slot),
         _ptr(batch.row_pos), _ptr(kv.page_table), _i(kv.page_table.shape[1]), _ptr(kv.keys), _ptr(kv.values),
         _i(_dtype_code(kv.keys)), _i(kv.page_size), _ptr(q_out), _i(_dtype_code(q_out)), _i(rows), _i(nq), _i(nkv), _i(d), _i(vd),
-        _stream()), "heads_prepare")
+        _i(maps), _stream()), "heads_prepare")
+
+
+def differential_output(a, lam, factor, eps, gate, out, H, V):
+    """``out[r, h] = rms(a[r, 2h] - lam a[r, 2h + 1]) * factor * sigmoid(gate[r, h])`` (heads of ``V``; ``gate``: float32 columns of a
+    matrix, or None)."""
+    _need_cuda(a, out)
+    rows = a.shape[0]
+    require(a.dtype == torch.float32 and a.shape == (rows, 2 * H * V) and out.shape == (rows, H * V)
+            and (gate is None or (gate.is_cuda and gate.dtype == torch.float32 and gate.shape == (rows, H) and gate.stride(1) == 1)),
+            "differential_output: shapes or dtypes do not fit")
+    _check(lib().citlali_differential_output(_ptr(a), _f(lam), _f(factor), _f(eps), _ptr(gate),
+                                             _sz(gate.stride(0) if gate is not None else 0), _ptr(out), _i(_dtype_code(out)), _i(rows),
+                                             _i(H), _i(V), _stream()), "differential_output")
 
 
 def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scale, softcap=0.0, gate=None, sink=None,
@@ -883,10 +923,11 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
     token (and no first tokens are kept), the prompt kernel otherwise; the 32-bit path and other sizes run the kernel whose
     launch depends on the row count alone.  ``softcap`` c > 0:
     the scaled scores become c tanh(s / c).  ``sink``, ``turns``, ``turn_pairs``: see :func:`attention_prefill`.  ``gate``: float32 columns of a matrix (a view whose rows may be further apart
-    than they are long), the output is multiplied by their sigmoids element by element."""
+    than they are long), the output is multiplied by their sigmoids element by element.  A float32 ``out`` behind bfloat16 queries
+    receives the result unrounded."""
     _need_cuda(q, kv.keys, kv.values, kv.page_table, out, sink, turns)
     rows = q.shape[0]
-    require(q.shape == (rows, nq * d) and out.shape == (rows, nq * vd) and q.dtype == out.dtype,
+    require(q.shape == (rows, nq * d) and out.shape == (rows, nq * vd) and out.dtype in (q.dtype, torch.float32),
             "attention_window: shapes or dtypes do not fit")
     _check_sink_and_turns(sink, turns, nq, rows, vd)
     gate_stride = 0
@@ -925,7 +966,55 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
         _ptr(q), _i(_dtype_code(q)), _ptr(kv.keys), _ptr(kv.values), _i(_dtype_code(kv.keys)), _ptr(kv.page_table),
         _i(kv.page_table.shape[1]), _ptr(batch.row_slot), _ptr(batch.row_pos), _ptr(out), _i(rows), _i(nq), _i(nkv), _i(d),
         _i(vd), _i(kv.page_size), _i(int(window or 0)), _i(int(keep_first or 0)), _i(max_keys), _f(scale), _f(softcap),
-        _ptr(gate), _sz(gate_stride), _ptr(sink), _ptr(turns), _i(1 if turn_pairs else 0), _stream()), "attention_window")
+        _ptr(gate), _sz(gate_stride), _ptr(sink), _ptr(turns), _i(1 if turn_pairs else 0),
+        _ptr(out if out.dtype != q.dtype else None), _stream()), "attention_window")
+
+
+# ---- memories that are decayed sums of outer products ---------------------------------------------------------------
+
+MEMORY_SCAN, MEMORY_SINGLE, MEMORY_CHUNKS = 0, 1, 2
+
+
+def memory_gates(zi, zf, bi, bf, cap, state, max_off, batch, logs, floors):
+    """``zi``, ``zf``: float32 columns [rows, H] of one matrix; see ``citlali_memory_gates``."""
+    _need_cuda(state, bi, bf, logs, floors)
+    rows, H = floors.shape
+    require(all(t.is_cuda and t.dtype == torch.float32 and t.shape == (rows, H) and t.stride(1) == 1 for t in (zi, zf))
+            and zi.stride(0) == zf.stride(0) and logs.shape == (rows, H, 2) and state.shape[1] >= max_off + H
+            and all(t.dtype == torch.float32 for t in (state, logs, floors)), "memory_gates: shapes or dtypes do not fit")
+    _check(lib().citlali_memory_gates(_ptr(zi), _ptr(zf), _sz(zi.stride(0)), _ptr(bi), _ptr(bf), _f(cap), _ptr(state), _sz(state.shape[1]),
+                                      _sz(max_off), _ptr(batch.seq_start), _ptr(batch.seq_slot), _i(batch.sequences), _i(H), _ptr(logs),
+                                      _ptr(floors), _stream()), "memory_gates")
+
+
+def linear_memory(q, k, v, state, batch, H, D, V, out, decay=None, logs=None, sums=None, sum_off=0, act=None, q_scale=1.0,
+                  form=MEMORY_SCAN):
+    """``q``, ``k`` [rows, H D] and ``v`` [rows, H V]: float32 columns of one matrix; see ``citlali_linear_memory``.  ``act``: None or
+    "silu"."""
+    _need_cuda(state, decay, logs, sums, out)
+    rows = out.shape[0]
+    require(all(t.is_cuda and t.dtype == torch.float32 and t.shape == (rows, H * n) and t.stride(1) == 1 and t.stride(0) == q.stride(0)
+                for t, n in ((q, D), (k, D), (v, V))) and out.shape == (rows, H * V) and out.dtype == torch.float32
+            and state.dtype == torch.float32 and state.shape[1] >= H * D * V and (sums is None or state.shape[1] >= sum_off + H * D)
+            and (decay is None or (decay.dtype == torch.float32 and decay.numel() == H))
+            and (logs is None or (logs.dtype == torch.float32 and logs.shape == (rows, H, 2))) and act in (None, "silu"),
+            "linear_memory: shapes or dtypes do not fit")
+    _check(lib().citlali_linear_memory(_ptr(q), _ptr(k), _ptr(v), _sz(q.stride(0)), _i(1 if act else 0), _f(q_scale), _ptr(decay),
+                                       _ptr(logs), _ptr(state), _sz(state.shape[1]), _sz(sum_off), _ptr(batch.seq_start),
+                                       _ptr(batch.seq_slot), _i(batch.sequences), _i(H), _i(D), _i(V), _ptr(out), _ptr(sums), _i(form),
+                                       _stream()), "linear_memory")
+
+
+def linear_memory_output(o, sums, floors, gate, weight, y, H, V, groups, eps):
+    """``gate``: float32 columns [rows, H V] of a matrix."""
+    _need_cuda(o, sums, floors, weight, y)
+    rows = o.shape[0]
+    require(o.dtype == torch.float32 and o.shape == y.shape == (rows, H * V) and gate.is_cuda and gate.dtype == torch.float32
+            and gate.shape == (rows, H * V) and gate.stride(1) == 1 and weight.dtype == torch.float32 and weight.numel() == H * V,
+            "linear_memory_output: shapes or dtypes do not fit")
+    _check(lib().citlali_linear_memory_output(_ptr(o), _ptr(sums), _ptr(floors), _ptr(gate), _sz(gate.stride(0)), _ptr(weight), _ptr(y),
+                                              _i(_dtype_code(y)), _i(rows), _i(H), _i(V), _i(groups), _f(eps), _stream()),
+           "linear_memory_output")
 
 
 # ---- routed experts -----------------------------------------------------------------------------------------------
@@ -933,10 +1022,15 @@ def attention_window(q, kv, batch, out, nq, nkv, d, vd, window, keep_first, scal
 ROUTER_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 
 
-def moe_route(logits, weights, groups, keep, top, chosen=None, weight_scale=1.0, score="softmax", bias=None, extra=None):
+def moe_route(logits, weights, groups, keep, top, chosen=None, weight_scale=1.0, score="softmax", bias=None, extra=None,
+              correction=None, group_best=1, renormalise=False):
     """``bias``: float32, a number an expert added to the logits.  ``extra`` float32 [rows]: receives the sigmoid of the one
-    column that ``logits`` has behind the experts'."""
-    _need_cuda(logits, weights, chosen, bias, extra)
+    column that ``logits`` has behind the experts'.  ``correction``: float32, a number an expert added to the scores for every
+    choice and not to the weights; ``group_best`` 2: a group's score is the sum of its two largest; ``renormalise``: the chosen
+    weights are divided by their sum ahead of ``weight_scale``."""
+    _need_cuda(logits, weights, chosen, bias, extra, correction)
+    require(correction is None or (correction.dtype == torch.float32 and correction.numel() == weights.shape[1]),
+            "moe_route: the correction does not fit")
     require(score in ROUTER_SCORES, f"moe_route: unknown score '{score}'; known: {', '.join(ROUTER_SCORES)}")
     rows, E = weights.shape
     require(logits.dtype == torch.float32 and weights.dtype == torch.float32
@@ -945,8 +1039,8 @@ def moe_route(logits, weights, groups, keep, top, chosen=None, weight_scale=1.0,
             and (extra is None or (extra.dtype == torch.float32 and extra.numel() == rows)) and (chosen is None or (chosen.dtype == torch.int32 and chosen.shape == (rows, top))),
             "moe_route: shapes or dtypes do not fit")
     _check(lib().citlali_moe_route(_ptr(logits), _ptr(weights), _ptr(chosen), _i(rows), _i(E), _i(int(groups or 0)),
-                                   _i(int(keep or 0)), _i(top), _f(weight_scale), _i(ROUTER_SCORES[score]), _i(logits.shape[1]), _ptr(bias), _ptr(extra), _stream()),
-           "moe_route")
+                                   _i(int(keep or 0)), _i(top), _f(weight_scale), _i(ROUTER_SCORES[score]), _i(logits.shape[1]), _ptr(bias), _ptr(extra),
+                                   _ptr(correction), _i(int(group_best)), _i(1 if renormalise else 0), _stream()), "moe_route")
 
 
 def moe_scale(act, weights, ff):
@@ -980,6 +1074,19 @@ def expert_gate(gate_up, weights, act, E, ff, run, kind, limit=0.0, alpha=1.0, t
                                      _i(rows), _i(E), _i(ff), _i(run), _i(EXPERT_ACTIVATIONS[kind]), _f(limit), _f(alpha),
                                      _i(tail_ff), _i(tail_run), _f(tail_limit), _ptr(bias), _i(1 if weight_input else 0),
                                      _ptr(tail_weights), _stream()), "expert_gate")
+
+
+def expert_relu_squared(z, weights, act, E, ff, tail_ff=0, tail_weights=None):
+    """``act = weights max(z, 0)^2`` over [rows, E ff + tail_ff]: ``E`` experts without a gate, times the row's weight for each, and one
+    that every row uses, times ``tail_weights`` [rows] (None: 1)."""
+    _need_cuda(z, weights, act, tail_weights)
+    rows, n = act.shape
+    require(z.shape == act.shape and n == E * ff + tail_ff
+            and (E == 0 or (weights is not None and weights.dtype == torch.float32 and weights.shape == (rows, E)))
+            and (tail_weights is None or (tail_weights.dtype == torch.float32 and tail_weights.numel() == rows)),
+            "expert_relu_squared: shapes or dtypes do not fit")
+    _check(lib().citlali_expert_relu_squared(_ptr(z), _i(_dtype_code(z)), _ptr(weights), _ptr(act), _i(_dtype_code(act)), _i(rows), _i(E),
+                                             _i(ff), _i(tail_ff), _ptr(tail_weights), _stream()), "expert_relu_squared")
 
 
 def bias_xielu(z, bias, ap, an, out):

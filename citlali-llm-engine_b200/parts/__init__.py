@@ -26,3 +26,6 @@ from . import embedding, mixer_input   # what is added to embedding rows, what m
 from .embedding import HashedPairEmbedding
 from .mixer_input import ResidualConv
 from .norm import GroupedRMSNorm
+from . import differential, linear_memory   # two more built-in mixers
+from .differential import DifferentialAttention
+from .linear_memory import LinearMemoryMixer

@@ -320,6 +320,54 @@ class InputInjectionBlock:
         return x
 
 
+class InputAdditionBlock:
+    """x <- x + x0 + b_t: ahead of every pass over a run of layers that repeats but the first, the rows the embedding left (x0) are
+    added to the residual again, and ahead of every pass (the first too) a vector of its own, row t of a table ``[passes, hidden]``
+    (a schedule names the block once ahead of every pass).  32-bit; no cache.  If the block that runs next begins with a layer norm,
+    the same kernel runs it and leaves its rows for that block.  ``block_params``: hidden_size, passes, ``steps`` (the table's
+    full name)."""
+    graph_safe = True
+    kernel_sources = ("sublayer",)
+
+    def __init__(self, layer_spec):
+        bp = layer_spec.block_params
+        self.hidden, self.passes = int(bp["hidden_size"]), int(bp["passes"])
+        self.steps_name = str(bp["steps"])
+        self.needs_embedding_output = self.passes > 1
+
+    def parts(self):
+        return []
+
+    def tensor_specs(self):
+        return [TensorSpec(self.steps_name, (self.passes, self.hidden), "state")]
+
+    def cache_requirement(self):
+        return None
+
+    def bind(self, weights, ctx):
+        h = weights[self.steps_name]
+        require(tuple(h.shape) == (self.passes, self.hidden),
+                f"unexpected tensor shape for {self.steps_name}: got {list(h.shape)}, expected {[self.passes, self.hidden]}")
+        self.steps = h.tensor.to(device=ctx.device, dtype=torch.float32).contiguous()
+        self.dtype = ctx.dtype
+
+    def forward(self, x, batch, cache_view, write_cache=True):
+        require(0 <= batch.visit < self.passes, f"the input addition has run {batch.visit} times, its table has {self.passes} rows")
+        x0 = batch.embedding_output if batch.visit > 0 else None
+        require(batch.visit == 0 or (x0 is not None and x0.shape == x.shape and x0.data_ptr() != x.data_ptr()),
+                "the input addition needs the embedding's rows beside the residual")
+        nxt = batch.next_first_norm
+        if nxt is not None and callable(getattr(nxt, "chain_terms", None)) and nxt.size == self.hidden:
+            gain, bias, eps = nxt.chain_terms()
+            h = torch.empty(x.shape, dtype=self.dtype, device=x.device)
+            ops.add_rows_norm(x, x0, self.steps[batch.visit], gain, bias, eps, h)
+            batch.normed_carry = (h, nxt)
+        else:
+            ops.add_rows_norm(x, x0, self.steps[batch.visit])
+        return x
+
+
+register_part("block", "input_addition", InputAdditionBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)
 register_part("block", "input_injection", InputInjectionBlock)
 register_part("block", "pre_norm_residual", PreNormResidualBlock)

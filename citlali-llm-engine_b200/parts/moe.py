@@ -1,4 +1,4 @@
-"""Routed experts: a feed-forward made of ``experts`` small gated feed-forwards of which every token uses ``top``.
+"""Routed experts: a feed-forward made of ``experts`` small feed-forwards of which every token uses ``top``.
 
 Router logits z = W_router h in 32-bit; scores s = softmax(z) over all experts (``score`` "sigmoid": s = sigmoid(z), every
 expert's score by itself; "softmax_chosen": the logits choose, and the weights are the softmax over the chosen logits
@@ -24,9 +24,14 @@ activation), every expert's activations are multiplied by the row's weight for i
 by side are ONE product that sums over experts.  Nothing depends on counts known to the host
 only, so a decoding step replays as a graph; the price is that every expert's matrices are applied to every row.
 
+``activation`` "relu_squared" is for experts without a gate: W_down max(W_up h, 0)^2.  ``correction``: a number an expert is added to
+the scores wherever groups and experts are compared (the sums may be negative), not in the weights.  ``group_score`` "top2_sum": a
+group's score is the sum of its two largest scores (corrected, if they are).  ``renormalise``: the chosen weights are divided by
+their sum (+ 1e-20) ahead of ``weight_scale``.
+
 Parameters: hidden_size, experts, top, intermediate_size, groups, keep_groups, weight_scale, score, weight_on, activation,
-limit, alpha, shared, router_bias; ``names``: {"router": name, "router_bias": name, "gate": [names], "up": [names], "down":
-[names], "shared": {"gate", "up", "down", "weight"}} (default ``<prefix>.router``, ``<prefix>.router.b``,
+limit, alpha, shared, router_bias, correction, group_score, renormalise; ``names``: {"router": name, "router_bias": name, "correction": name, "gate": [names], "up": [names], "down":
+[names], "shared": {"gate", "up", "down", "weight"}} (default ``<prefix>.router``, ``<prefix>.router.b``, ``<prefix>.correction``,
 ``<prefix>.e<i>.{gate,up,down}``, ``<prefix>.shared.{gate,up,down}`` and ``<prefix>.shared.sg``).
 """
 from __future__ import annotations
@@ -62,8 +67,10 @@ class RoutedExperts:
         self.weight_input = {"output": False, "input": True}.get(str(params.get("weight_on") or "output"))
         require(self.weight_input is not None, f"{prefix}: weight_on must be 'output' or 'input'")
         self.activation = str(params.get("activation") or "silu")
-        require(self.activation in ops.EXPERT_ACTIVATIONS,
-                f"{prefix}: unknown expert activation '{self.activation}'; known: {', '.join(ops.EXPERT_ACTIVATIONS)}")
+        self.has_gate = self.activation != "relu_squared"
+        known = tuple(ops.EXPERT_ACTIVATIONS) + ("relu_squared",)
+        require(self.activation in known, f"{prefix}: unknown expert activation '{self.activation}'; known: {', '.join(known)}")
+        require(self.has_gate or not self.weight_input, f"{prefix}: experts without a gate weight their output")
         self.limit = float(params.get("limit") or 0.0)
         self.alpha = 1.702 if params.get("alpha") is None else float(params["alpha"])
         require(self.activation != "clamped_swish" or self.limit > 0.0, f"{prefix}: the clamped activation needs a positive limit")
@@ -74,7 +81,11 @@ class RoutedExperts:
         gate_up_tail = down_tail = None
         self.shared_weighted, router_names, router_sizes = False, [str(n.get("router") or f"{prefix}.router")], [self.E]
         self.router_bias_name = str(n.get("router_bias") or f"{prefix}.router.b") if params.get("router_bias") else None
-        self.router_bias = None
+        self.router_bias = self.correction = None
+        self.correction_name = str(n.get("correction") or f"{prefix}.correction") if params.get("correction") else None
+        self.group_best = {"max": 1, "top2_sum": 2}.get(str(params.get("group_score") or "max"))
+        require(self.group_best is not None, f"{prefix}: group_score must be 'max' or 'top2_sum'")
+        self.renormalise = bool(params.get("renormalise", False))
         if shared is not None:
             self.shared_ff = int(shared["intermediate_size"])
             self.shared_limit = float(shared.get("limit") or 0.0)
@@ -82,7 +93,7 @@ class RoutedExperts:
                     f"{prefix}: the expert for every row needs a width and, with the clamped activation, a positive limit")
             sn = dict(n.get("shared") or {})
             name = lambda role: str(sn.get(role) or f"{prefix}.shared.{role}")
-            gate_up_tail = (name("gate"), name("up"), self.shared_ff)
+            gate_up_tail = (name("gate"), name("up"), self.shared_ff) if self.has_gate else (name("up"), self.shared_ff)
             down_tail = (name("down"), self.shared_ff)
             require(shared.get("weight") in (None, "sigmoid"), f"{prefix}: the weight of the expert for every row is 'sigmoid' or None")
             self.shared_weighted = shared.get("weight") is not None
@@ -90,7 +101,11 @@ class RoutedExperts:
                 router_names.append(str(sn.get("weight") or f"{prefix}.shared.sg"))
                 router_sizes.append(1)
         self.router = DenseLinear(router_names, router_sizes, self.hidden)
-        self.gate_up = ExpertGateUp(each("gate"), each("up"), self.ff, self.hidden, tail=gate_up_tail)
+        if self.has_gate:
+            self.gate_up = ExpertGateUp(each("gate"), each("up"), self.ff, self.hidden, tail=gate_up_tail)
+        else:                    # the up matrices of all experts, one below the other
+            tail = gate_up_tail or ()
+            self.gate_up = DenseLinear(each("up") + list(tail[:1]), [self.ff] * self.E + list(tail[1:]), self.hidden)
         self.down = ExpertDown(each("down"), self.ff, self.hidden, tail=down_tail)
         self.prefix = prefix
         # the product's own gate epilogue and the scaling kernel serve the plain form; anything else runs the gate kernel
@@ -98,6 +113,8 @@ class RoutedExperts:
 
     def tensor_specs(self):
         bias = [TensorSpec(self.router_bias_name, (self.E,), "state")] if self.router_bias_name is not None else []
+        if self.correction_name is not None:
+            bias.append(TensorSpec(self.correction_name, (self.E,), "state"))
         return self.router.tensor_specs() + bias + self.gate_up.tensor_specs() + self.down.tensor_specs()
 
     def bind(self, weights, ctx):
@@ -106,6 +123,8 @@ class RoutedExperts:
         self.down.bind(weights, ctx)
         if self.router_bias_name is not None:
             self.router_bias = bind_vector(weights, self.router_bias_name, self.E, ctx)
+        if self.correction_name is not None:
+            self.correction = bind_vector(weights, self.correction_name, self.E, ctx)
         self.dtype = ctx.dtype
 
     def route(self, h):
@@ -118,12 +137,17 @@ class RoutedExperts:
         weights = torch.empty((h.shape[0], self.E), dtype=torch.float32, device=h.device)
         extra = torch.empty((h.shape[0],), dtype=torch.float32, device=h.device) if self.shared_weighted else None
         ops.moe_route(logits, weights, self.groups, self.keep, self.top, weight_scale=self.weight_scale, score=self.score,
-                      bias=self.router_bias, extra=extra)
+                      bias=self.router_bias, extra=extra, correction=self.correction, group_best=self.group_best,
+                      renormalise=self.renormalise)
         return weights, extra
 
     def forward(self, h, batch, residual, overwrite=False):
         weights, extra = self._route(h)
-        if self.plain:
+        if not self.has_gate:
+            z = self.gate_up.forward(h, out_dtype=torch.float32)
+            act = torch.empty((h.shape[0], self.E * self.ff + self.shared_ff), dtype=self.dtype, device=h.device)
+            ops.expert_relu_squared(z, weights, act, self.E, self.ff, self.shared_ff, tail_weights=extra)
+        elif self.plain:
             act = self.gate_up.forward_gated(h, self.gate_up.run)
             if act is None:
                 act = torch.empty((h.shape[0], self.E * self.ff), dtype=self.dtype, device=h.device)

@@ -85,7 +85,8 @@ class LayerNorm:
     rows in the compute dtype; ``chain_terms`` gives a block what it needs to run this norm inside a kernel of its own.
 
     Parameters: size, eps; optional ``tensor`` (the gain's full name; default ``<prefix>.weight``) and ``bias`` (the bias's
-    full name; None: no bias).  A norm with a bias keeps gain and bias in float32 in both paths."""
+    full name; None: no bias), ``scale`` (the result is multiplied by it: gain and bias are, once, in float32).  A norm with a bias
+    or a scale keeps gain and bias in float32 in both paths."""
     graph_safe = True
     kernel_sources = ("sublayer",)
 
@@ -94,6 +95,7 @@ class LayerNorm:
         self.eps = float(params["eps"])
         self.name = str(params.get("tensor") or f"{prefix}.weight")
         self.bias_name = None if params.get("bias") is None else str(params["bias"])
+        self.scale = 1.0 if params.get("scale") is None else float(params["scale"])
         self.gain = self.bias = None
 
     def tensor_specs(self):
@@ -103,11 +105,12 @@ class LayerNorm:
         return specs
 
     def bind(self, weights, ctx):
-        if self.bias_name is None:
+        if self.bias_name is None and self.scale == 1.0:
             self.gain = bind_gain(weights, self.name, self.size, ctx)
         else:
-            self.gain = bind_vector(weights, self.name, self.size, ctx)
-            self.bias = bind_vector(weights, self.bias_name, self.size, ctx)
+            self.gain = bind_vector(weights, self.name, self.size, ctx) * self.scale
+            if self.bias_name is not None:
+                self.bias = bind_vector(weights, self.bias_name, self.size, ctx) * self.scale
         self.dtype = ctx.dtype
 
     def forward(self, x: torch.Tensor, row_index=None) -> torch.Tensor:
