@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
     python bench.py --workload 3|4 [--repetitions R]      the batch workloads of BASELINE.json's other shapes
-    python bench.py --design lanizen|gidirax|sobunex|pivavik|nomutar [--sizes small,medium,large]   a design beside another at equal size
+    python bench.py --design lanizen|gidirax|sobunex|pivavik|nomutar|kopalorn [--sizes small,medium,large]   a design beside another at equal size
 
 Prints ONE JSON line.  For each batch size (8, and 1 and 64 unless --skip-points) the run is a real one: the
 prompts (2,048 random tokens each) are prefilled in one step, then every sequence is decoded token by token up
@@ -366,7 +366,7 @@ def main():
     ap.add_argument("--run-from", type=int, default=None,
                     help="length of the prompts of the decode runs (default: the prefill length, 2,048); close to the context "
                          "length it makes a short run, as a profiler capture needs")
-    ap.add_argument("--design", default=None, choices=["lanizen", "gidirax", "sobunex", "pivavik", "nomutar"],
+    ap.add_argument("--design", default=None, choices=["lanizen", "gidirax", "sobunex", "pivavik", "nomutar", "kopalorn"],
                     help="measure this design beside the library's closest other design at equal sizes (prompt step, decode "
                          "step, every kernel of both) instead of the benchmark configuration")
     ap.add_argument("--sizes", default="medium,large", help="with --design: which of small, medium, large")

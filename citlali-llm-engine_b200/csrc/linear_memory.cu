@@ -60,14 +60,27 @@ memory_gates_kernel(const float* __restrict__ zi, const float* __restrict__ zf, 
     float* slot = state + (size_t)seq_slot[seq] * state_stride + max_off + h;
     const float b_i = bi ? bi[h] : 0.0f, b_f = bf ? bf[h] : 0.0f;
     float m = *slot;
-    for (int base = r0; base < r1; base += 32) {             // a lane a token; the maxima in order
+    constexpr int AHEAD = 4;                                  // runs of 32 tokens whose inputs are on their way
+    float next_i[AHEAD], next_f[AHEAD];
+    auto fetch = [&](int base, int j) {
+        const int row = base + lane;
+        if (row < r1) { next_i[j] = zi[row * stride + h]; next_f[j] = zf[row * stride + h]; }
+    };
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) fetch(r0 + 32 * j, j);
+    for (int group = r0; group < r1; group += 32 * AHEAD)
+#pragma unroll
+    for (int g = 0; g < AHEAD; ++g) {                        // a lane a token; the maxima in order
+        const int base = group + 32 * g;
+        if (base >= r1) break;
         const int row = base + lane, n = min(32, r1 - base);
         float i = 0.0f, f = 0.0f;
         if (row < r1) {
-            i = cap * tanhf((zi[row * stride + h] + b_i) / cap);
-            const float z = cap * tanhf((zf[row * stride + h] + b_f) / cap);
+            i = cap * tanhf((next_i[g] + b_i) / cap);
+            const float z = cap * tanhf((next_f[g] + b_f) / cap);
             f = fminf(z, 0.0f) - log1pf(expf(-fabsf(z)));
         }
+        fetch(base + 32 * AHEAD, g);
         float before = 0.0f, after = 0.0f;
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
@@ -197,12 +210,15 @@ linear_memory_scan_kernel(MemoryArgs a) {
 //   S  <- exp(A_63) S + sum_s exp(A_63 - A_s + w_s) k_s v_s^T.
 // All exponents are at most zero.  The products run as mma.sync m16n8k16: bfloat16 operands (S as the sum of two bfloat16
 // numbers, so that it enters with 16 bits of mantissa), float32 sums.  S stays in float32 accumulators from chunk to chunk;
-// exponents and their sums are float32.  Eight warps: warps w and w + 4 share the chunk's tokens 16 w .. 16 w + 15 and the
-// rows D/4 w .. of S; the first takes columns 0-15 (and the key sum, as one more column whose v is 1), the second 16-31.
-constexpr int kChunk = 64, kCols = 32, kTileCols = 48, kColPitch = 56;     // columns a block, of a tile in shared memory, its pitch
+// exponents and their sums are float32.  Sixteen warps: warp (band, quarter) makes the weights of tokens 16 band .. + 15 for the
+// keys 16 quarter .. + 15 (shared memory passes them on, rounded), and of those tokens' results and of the rows D/4 band .. of S
+// the columns 8 quarter .. + 7; the first quarter also takes the key sum, as one more column whose v is 1.
+constexpr int kChunk = 64, kCols = 32, kColPitch = 56, kWeightPitch = 72;  // columns a block; pitches of tiles in shared memory
+constexpr int kChunkThreads = 512;
 
-template <int DP>
-__global__ void __launch_bounds__(256)
+// VEC: sizes and strides are multiples of four and addresses of 16 bytes.
+template <int DP, bool VEC>
+__global__ void __launch_bounds__(kChunkThreads, 1)
 linear_memory_chunks_kernel(MemoryArgs a) {
     using namespace fa;
     constexpr int PITCH = DP + 8, MT = DP / 64;
@@ -213,10 +229,11 @@ linear_memory_chunks_kernel(MemoryArgs a) {
     __nv_bfloat16* sw = sv + kChunk * kColPitch;                             // the same times exp(A_63 - A_s + w_s)
     __nv_bfloat16* s_hi = sw + kChunk * kColPitch;                           // [DP][kColPitch] S, rounded
     __nv_bfloat16* s_lo = s_hi + DP * kColPitch;                             // and what the rounding left
+    __nv_bfloat16* sp = s_lo + DP * kColPitch;                               // [64][kWeightPitch] the chunk's weights
     __shared__ float sum_a[kChunk], from[kChunk], share[kChunk];             // A_t, w_s - A_s, exp(A_63 - A_s + w_s); in log2 units
     dependents_may_launch();
     wait_for_predecessor();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, band = warp & 3, half = warp >> 2;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, band = warp & 3, quarter = warp >> 2;
     const int D = a.D, V = a.V, slices = (V + kCols - 1) / kCols;
     const int slice = blockIdx.x % slices, head = (blockIdx.x / slices) % a.H, seq = blockIdx.x / (slices * a.H);
     const int col0 = slice * kCols;
@@ -225,31 +242,30 @@ linear_memory_chunks_kernel(MemoryArgs a) {
     float* region = a.state + (size_t)a.seq_slot[seq] * a.state_stride;
     float* S_g = region + (size_t)head * D * V;
     float* n_g = region + a.sum_off + (size_t)head * D;
-    const int tiles = (half == 0 && with_sum) ? 3 : 2;                       // column tiles of eight this warp works on
-    auto tile_col = [&](int j) { return j == 2 ? kCols : half * 16 + j * 8; };
+    const int tiles = (quarter == 0 && with_sum) ? 2 : 1;                    // column tiles of eight this warp works on
+    auto tile_col = [&](int j) { return j == 1 ? kCols : quarter * 8; };
     // element (i, e) of an accumulator: row lane/4 (+ 8 for e >= 2), column (lane % 4) * 2 + e % 2
     auto place = [&](int m, int j, int e) -> float* {
         const int d = (band * MT + m) * 16 + (lane >> 2) + (e >> 1) * 8, c = tile_col(j) + (lane & 3) * 2 + (e & 1);
         if (d >= D) return nullptr;
-        if (j == 2) return c == kCols ? n_g + d : nullptr;
+        if (j == 1) return c == kCols ? n_g + d : nullptr;
         return col0 + c < V ? S_g + (size_t)d * V + col0 + c : nullptr;
     };
-    float S[MT][3][4];
+    float S[MT][2][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int j = 0; j < 3; ++j)
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const float* p = j < tiles ? place(m, j, e) : nullptr;
                 S[m][j][e] = p ? *p : 0.0f;
             }
     const float log_keep = a.decay ? (a.decay[head] > 0.0f ? log2f(a.decay[head]) : -1e30f) : 0.0f;   // (a decay of zero: finite, 64 of them too)
-    const bool vec = D % 4 == 0 && V % 4 == 0 && a.stride % 4 == 0 && (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15u) == 0;
-    // four neighbouring elements of a row, zeros past `limit`, through the activation
-    auto fetch = [&](const float* row, int c, int limit, float scale) -> uint2 {
+    // four neighbouring elements of a row as they are (zeros past `limit`), and through the activation as two words
+    auto fetch = [&](const float* row, int c, int limit) -> float4 {
         float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (vec) {
+        if constexpr (VEC) {
             if (c < limit) x = *reinterpret_cast<const float4*>(row + c);
         } else {
             if (c < limit) x.x = row[c];
@@ -257,15 +273,74 @@ linear_memory_chunks_kernel(MemoryArgs a) {
             if (c + 2 < limit) x.z = row[c + 2];
             if (c + 3 < limit) x.w = row[c + 3];
         }
+        return x;
+    };
+    auto words = [&](float4 x) -> uint2 {
         if (a.act) {
             x.x = __fdividef(x.x, 1.0f + __expf(-x.x)); x.y = __fdividef(x.y, 1.0f + __expf(-x.y));
             x.z = __fdividef(x.z, 1.0f + __expf(-x.z)); x.w = __fdividef(x.w, 1.0f + __expf(-x.w));
         }
-        return make_uint2(pack_bf16(x.x * scale, x.y * scale), pack_bf16(x.z * scale, x.w * scale));
+        return make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
     };
+    // a thread's pieces of the chunk's rows: q and k of up to 128 elements, and v, wait in registers while the chunk before is
+    // worked on; wider heads fetch half of their pieces at a time when the tiles are filled
+    constexpr int PIECES = kChunk * (DP / 4) / kChunkThreads;
+    static_assert(kChunk * (kCols / 4) == kChunkThreads && PIECES >= 1, "a piece of v a thread");
+    constexpr bool AHEAD = DP <= 128;
+    constexpr int HELD = AHEAD ? PIECES : PIECES / 2;
+    float4 rq[HELD], rk[HELD], rv;
+    const int v_row = tid / (kCols / 4), v_col = tid % (kCols / 4) * 4;
+    const size_t chunk_step = (size_t)kChunk * a.stride;
+    const float* v_next = a.v + (size_t)(r0 + v_row) * a.stride + (size_t)head * V;
+    constexpr int ROWS_APART = AHEAD ? kChunkThreads / (DP / 4) : 1;          // rows from one of a thread's pieces to the next
+    const int q_row = tid / (DP / 4), q_col = tid % (DP / 4) * 4;
+    const float* q_next = a.q + (size_t)(r0 + q_row) * a.stride + (size_t)head * D;
+    const float* k_next = a.k + (size_t)(r0 + q_row) * a.stride + (size_t)head * D;
+    auto fetch_next_qk = [&](int t0) {
+#pragma unroll
+        for (int i = 0; i < HELD; ++i) {
+            const int limit = t0 + q_row + i * ROWS_APART < n ? D : 0;
+            rq[i] = fetch(q_next + (size_t)(i * ROWS_APART) * a.stride, q_col, limit);
+            rk[i] = fetch(k_next + (size_t)(i * ROWS_APART) * a.stride, q_col, limit);
+        }
+        q_next += chunk_step;
+        k_next += chunk_step;
+    };
+    auto fetch_qk = [&](int t0, int first) {
+#pragma unroll
+        for (int i = 0; i < HELD; ++i) {
+            const int at = tid + (first + i) * kChunkThreads, t = at / (DP / 4), c = at % (DP / 4) * 4;
+            const size_t row = (size_t)(r0 + t0 + t) * a.stride + (size_t)head * D;
+            const int limit = t0 + t < n ? D : 0;
+            rq[i] = fetch(a.q + row, c, limit);
+            rk[i] = fetch(a.k + row, c, limit);
+        }
+    };
+    auto store_qk = [&](int first) {
+#pragma unroll
+        for (int i = 0; i < HELD; ++i) {
+            const int at = tid + (first + i) * kChunkThreads, t = at / (DP / 4), c = at % (DP / 4) * 4;
+            *reinterpret_cast<uint2*>(sq + t * PITCH + c) = words(rq[i]);
+            *reinterpret_cast<uint2*>(sk + t * PITCH + c) = words(rk[i]);
+        }
+    };
+    auto fetch_v = [&](int t0) {
+        rv = fetch(v_next, col0 + v_col, t0 + v_row < n ? V : 0);
+        v_next += chunk_step;
+    };
+    float2 next_log[2];
+    auto fetch_logs = [&](int t0) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+            if (!a.decay && t0 + 2 * lane + e < n) next_log[e] = a.logs[(size_t)(r0 + t0 + 2 * lane + e) * a.H + head];
+    };
+    if (warp == 0) fetch_logs(0);
+    if constexpr (AHEAD) fetch_next_qk(0);
+    fetch_v(0);
     const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(sq), k_addr = (uint32_t)__cvta_generic_to_shared(sk);
     const uint32_t v_addr = (uint32_t)__cvta_generic_to_shared(sv), w_addr = (uint32_t)__cvta_generic_to_shared(sw);
     const uint32_t hi_addr = (uint32_t)__cvta_generic_to_shared(s_hi), lo_addr = (uint32_t)__cvta_generic_to_shared(s_lo);
+    const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(sp);
 
     for (int t0 = 0; t0 < n; t0 += kChunk) {
         const int here = min(kChunk, n - t0);
@@ -274,17 +349,11 @@ linear_memory_chunks_kernel(MemoryArgs a) {
             float keep[2], write[2];
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const int t = 2 * lane + e;
-                keep[e] = 0.0f; write[e] = 0.0f;
-                if (t < here) {
-                    if (a.decay) {
-                        keep[e] = log_keep;
-                    } else {
-                        const float2 l = a.logs[(size_t)(r0 + t0 + t) * a.H + head];
-                        keep[e] = l.x * kLog2e; write[e] = l.y * kLog2e;
-                    }
-                }
+                const bool on = 2 * lane + e < here;
+                keep[e] = on ? (a.decay ? log_keep : next_log[e].x * kLog2e) : 0.0f;
+                write[e] = on && !a.decay ? next_log[e].y * kLog2e : 0.0f;
             }
+            fetch_logs(t0 + kChunk);
             float run = keep[0] + keep[1];
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -302,7 +371,7 @@ linear_memory_chunks_kernel(MemoryArgs a) {
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int j = 0; j < 3; ++j)
+            for (int j = 0; j < 2; ++j)
                 if (j < tiles) {
 #pragma unroll
                     for (int e = 0; e < 4; e += 2) {
@@ -314,141 +383,139 @@ linear_memory_chunks_kernel(MemoryArgs a) {
                     }
                 }
         // the chunk's rows
-        for (int i = tid; i < kChunk * (DP / 4); i += 256) {
-            const int t = i / (DP / 4), c = i % (DP / 4) * 4;
-            uint2 qw = make_uint2(0u, 0u), kw = make_uint2(0u, 0u);
-            if (t < here && c < D) {
-                const size_t at = (size_t)(r0 + t0 + t) * a.stride + (size_t)head * D;
-                qw = fetch(a.q + at, c, D, a.q_scale);
-                kw = fetch(a.k + at, c, D, 1.0f);
+        if constexpr (AHEAD) {
+            store_qk(0);
+            if (t0 + kChunk < n) fetch_next_qk(t0 + kChunk);  // on its way while this chunk is worked on
+        } else {
+#pragma unroll 1
+            for (int first = 0; first < PIECES; first += HELD) {
+                fetch_qk(t0, first);
+                store_qk(first);
             }
-            *reinterpret_cast<uint2*>(sq + t * PITCH + c) = qw;
-            *reinterpret_cast<uint2*>(sk + t * PITCH + c) = kw;
         }
-        __syncthreads();                         // (the shares are there)
-        for (int i = tid; i < kChunk * (kTileCols / 4); i += 256) {
-            const int t = i / (kTileCols / 4), c = i % (kTileCols / 4) * 4;
-            uint2 vw = make_uint2(0u, 0u);
-            if (t < here) {
-                if (c < kCols) {
-                    if (col0 + c < V) vw = fetch(a.v + (size_t)(r0 + t0 + t) * a.stride + (size_t)head * V, col0 + c, V, 1.0f);
-                } else if (c == kCols) {
-                    vw.x = pack_bf16(1.0f, 0.0f);
-                }
-            }
-            *reinterpret_cast<uint2*>(sv + t * kColPitch + c) = vw;
-            const float f = share[t];
+        __syncthreads();                         // (q, k, the state and the shares are there)
+        {
+            const uint2 vw = words(rv);
+            *reinterpret_cast<uint2*>(sv + v_row * kColPitch + v_col) = vw;
+            const float f = share[v_row];
             const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vw.x));
             const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vw.y));
-            *reinterpret_cast<uint2*>(sw + t * kColPitch + c) = make_uint2(pack_bf16(lo.x * f, lo.y * f), pack_bf16(hi.x * f, hi.y * f));
+            *reinterpret_cast<uint2*>(sw + v_row * kColPitch + v_col) = make_uint2(pack_bf16(lo.x * f, lo.y * f), pack_bf16(hi.x * f, hi.y * f));
+            if (t0 + kChunk < n) fetch_v(t0 + kChunk);
         }
-        __syncthreads();
-        // o of this warp's sixteen tokens: first S^T q, then scaled, then the chunk's own tokens
-        float o[3][4], p[kChunk / 8][4];
+        if (with_sum && tid < kChunk) {          // the key sum's column of ones, and seven of zeros
+            *reinterpret_cast<uint4*>(sv + tid * kColPitch + kCols) = make_uint4(tid < here ? 0x3f80u : 0u, 0u, 0u, 0u);
+            *reinterpret_cast<uint4*>(sw + tid * kColPitch + kCols) = make_uint4(pack_bf16(share[tid], 0.0f), 0u, 0u, 0u);
+        }
+        // S^T q of this warp's tokens and columns, and its sixteen by sixteen weights of the chunk's own tokens
+        float o[2][4], p[2][4];
 #pragma unroll
-        for (int j = 0; j < 3; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
-#pragma unroll
-        for (int i = 0; i < kChunk / 8; ++i) p[i][0] = p[i][1] = p[i][2] = p[i][3] = 0.0f;
+        for (int j = 0; j < 2; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = p[j][0] = p[j][1] = p[j][2] = p[j][3] = 0.0f;
         const int arow = band * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, acol = (lane >> 4) * 8;
-        const int brow = (lane & 7) + ((lane >> 3) & 1) * 8, bcol = (lane >> 4) * 8;
-        if (band * 16 < here) {
+        const int t_a = band * 16 + (lane >> 2), t_b = t_a + 8;
+        const bool rows_here = band * 16 < here, seen = quarter <= band;      // (later tokens are not seen)
+        if (rows_here) {
+            const uint32_t half_addr = (lane >> 4) ? lo_addr : hi_addr;       // one load brings both parts of sixteen rows of S
 #pragma unroll
             for (int ks = 0; ks < DP / 16; ++ks) {
                 uint32_t q0, q1, q2, q3, b0, b1, b2, b3;
                 ldmatrix_x4(q_addr + (arow * PITCH + ks * 16 + acol) * 2, q0, q1, q2, q3);
 #pragma unroll
-                for (int part = 0; part < 2; ++part) {
-                    const uint32_t base = (part ? lo_addr : hi_addr) + (ks * 16 + brow) * kColPitch * 2;
-                    ldmatrix_x4_trans(base + (half * 16 + bcol) * 2, b0, b1, b2, b3);
-                    mma_16816(o[0], q0, q1, q2, q3, b0, b1);
-                    mma_16816(o[1], q0, q1, q2, q3, b2, b3);
-                    if (tiles == 3) {
-                        ldmatrix_x4_trans(base + (kCols + bcol) * 2, b0, b1, b2, b3);
-                        mma_16816(o[2], q0, q1, q2, q3, b0, b1);
+                for (int j = 0; j < 2; ++j)
+                    if (j < tiles) {
+                        ldmatrix_x4_trans(half_addr + ((ks * 16 + (lane & 15)) * kColPitch + tile_col(j)) * 2, b0, b1, b2, b3);
+                        mma_16816(o[j], q0, q1, q2, q3, b0, b1);
+                        mma_16816(o[j], q0, q1, q2, q3, b2, b3);
                     }
-                }
-#pragma unroll
-                for (int np = 0; np < kChunk / 16; ++np) {
-                    if (np > band) break;                    // later tokens are not seen
-                    const int r = np * 16 + (lane & 7) + (lane >> 4) * 8, c = ((lane >> 3) & 1) * 8;
+                if (seen) {
+                    const int r = quarter * 16 + (lane & 7) + (lane >> 4) * 8, c = ((lane >> 3) & 1) * 8;
                     ldmatrix_x4(k_addr + (r * PITCH + ks * 16 + c) * 2, b0, b1, b2, b3);
-                    mma_16816(p[2 * np], q0, q1, q2, q3, b0, b1);
-                    mma_16816(p[2 * np + 1], q0, q1, q2, q3, b2, b3);
+                    mma_16816(p[0], q0, q1, q2, q3, b0, b1);
+                    mma_16816(p[1], q0, q1, q2, q3, b2, b3);
                 }
             }
-            const int t_a = band * 16 + (lane >> 2), t_b = t_a + 8;
-            const float A_a = sum_a[t_a], A_b = sum_a[t_b], g_a = exp2f(A_a), g_b = exp2f(A_b);
+            const float A_a = sum_a[t_a], A_b = sum_a[t_b], g_a = exp2f(A_a) * a.q_scale, g_b = exp2f(A_b) * a.q_scale;
 #pragma unroll
-            for (int j = 0; j < 3; ++j) { o[j][0] *= g_a; o[j][1] *= g_a; o[j][2] *= g_b; o[j][3] *= g_b; }
+            for (int j = 0; j < 2; ++j) { o[j][0] *= g_a; o[j][1] *= g_a; o[j][2] *= g_b; o[j][3] *= g_b; }
+            if (seen) {
 #pragma unroll
-            for (int np = 0; np < kChunk / 16; ++np) {
+                for (int i = 0; i < 2; ++i) {
+                    const int s = quarter * 16 + i * 8 + (lane & 3) * 2;
+                    const float f0 = from[s], f1 = from[s + 1];
+                    const float w0 = s <= t_a ? p[i][0] * (a.q_scale * exp2f(A_a + f0)) : 0.0f, w1 = s + 1 <= t_a ? p[i][1] * (a.q_scale * exp2f(A_a + f1)) : 0.0f;
+                    const float w2 = s <= t_b ? p[i][2] * (a.q_scale * exp2f(A_b + f0)) : 0.0f, w3 = s + 1 <= t_b ? p[i][3] * (a.q_scale * exp2f(A_b + f1)) : 0.0f;
+                    *reinterpret_cast<uint32_t*>(sp + t_a * kWeightPitch + s) = pack_bf16(w0, w1);
+                    *reinterpret_cast<uint32_t*>(sp + t_b * kWeightPitch + s) = pack_bf16(w2, w3);
+                }
+            }
+        }
+        __syncthreads();                         // (weights and values are there)
+        if (rows_here) {
+#pragma unroll
+            for (int np = 0; np < kChunk / 16; np += 2) {
                 if (np > band) break;
+                uint32_t b[2][4];
 #pragma unroll
-                for (int i = 2 * np; i < 2 * np + 2; ++i)
+                for (int j = 0; j < 2; ++j)
+                    if (j < tiles) ldmatrix_x4_trans(v_addr + ((np * 16 + lane) * kColPitch + tile_col(j)) * 2, b[j][0], b[j][1], b[j][2], b[j][3]);
 #pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const int s = i * 8 + (lane & 3) * 2 + e;
-                        const float f = from[s];
-                        p[i][e] = s <= t_a ? p[i][e] * exp2f(A_a + f) : 0.0f;
-                        p[i][e + 2] = s <= t_b ? p[i][e + 2] * exp2f(A_b + f) : 0.0f;
-                    }
-                const uint32_t p0 = pack_bf16(p[2 * np][0], p[2 * np][1]), p1 = pack_bf16(p[2 * np][2], p[2 * np][3]);
-                const uint32_t p2 = pack_bf16(p[2 * np + 1][0], p[2 * np + 1][1]), p3 = pack_bf16(p[2 * np + 1][2], p[2 * np + 1][3]);
-                const uint32_t base = v_addr + (np * 16 + brow) * kColPitch * 2;
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(base + (half * 16 + bcol) * 2, b0, b1, b2, b3);
-                mma_16816(o[0], p0, p1, p2, p3, b0, b1);
-                mma_16816(o[1], p0, p1, p2, p3, b2, b3);
-                if (tiles == 3) {
-                    ldmatrix_x4_trans(base + (kCols + bcol) * 2, b0, b1, b2, b3);
-                    mma_16816(o[2], p0, p1, p2, p3, b0, b1);
+                for (int i = 0; i < 2; ++i) {
+                    if (np + i > band) break;
+                    uint32_t p0, p1, p2, p3;
+                    ldmatrix_x4(p_addr + (arow * kWeightPitch + (np + i) * 16 + acol) * 2, p0, p1, p2, p3);
+#pragma unroll
+                    for (int j = 0; j < 2; ++j)
+                        if (j < tiles) mma_16816(o[j], p0, p1, p2, p3, b[j][2 * i], b[j][2 * i + 1]);
                 }
             }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int t = e < 2 ? t_a : t_b;
+            for (int e = 0; e < 4; e += 2) {
+                const int t = e < 2 ? t_a : t_b, c = col0 + quarter * 8 + (lane & 3) * 2;
                 if (t < here) {
                     const size_t row = r0 + t0 + t;
-#pragma unroll
-                    for (int j = 0; j < 2; ++j) {
-                        const int c = col0 + tile_col(j) + (lane & 3) * 2 + (e & 1);
-                        if (c < V) a.out[row * a.H * V + (size_t)head * V + c] = o[j][e];
+                    float* dst = a.out + row * a.H * V + (size_t)head * V + c;
+                    if (V % 2 == 0) {
+                        if (c < V) *reinterpret_cast<float2*>(dst) = make_float2(o[0][e], o[0][e + 1]);
+                    } else {
+                        if (c < V) dst[0] = o[0][e];
+                        if (c + 1 < V) dst[1] = o[0][e + 1];
                     }
-                    if (tiles == 3 && (lane & 3) == 0 && (e & 1) == 0) a.sums[row * a.H + head] = o[2][e];
+                    if (tiles == 2 && (lane & 3) == 0) a.sums[row * a.H + head] = o[1][e];
                 }
             }
         }
         // the state behind the chunk
         const float g = exp2f(sum_a[kChunk - 1]);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
+        for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int j = 0; j < 3; ++j) { S[m][j][0] *= g; S[m][j][1] *= g; S[m][j][2] *= g; S[m][j][3] *= g; }
-        }
+            for (int j = 0; j < 2; ++j) { S[m][j][0] *= g; S[m][j][1] *= g; S[m][j][2] *= g; S[m][j][3] *= g; }
 #pragma unroll
-        for (int kt = 0; kt < kChunk / 16; ++kt) {
+        for (int kt = 0; kt < kChunk / 16; kt += 2) {
             if (kt * 16 >= here) break;
-            uint32_t b0, b1, b2, b3, c0 = 0, c1 = 0, c2, c3;
-            const uint32_t base = w_addr + (kt * 16 + brow) * kColPitch * 2;
-            ldmatrix_x4_trans(base + (half * 16 + bcol) * 2, b0, b1, b2, b3);
-            if (tiles == 3) ldmatrix_x4_trans(base + (kCols + bcol) * 2, c0, c1, c2, c3);
+            uint32_t b[2][4];
 #pragma unroll
-            for (int m = 0; m < MT; ++m) {
-                // K^T: the tile lies as [token][d], its transpose is the operand
-                const int r = kt * 16 + (lane & 7) + (lane >> 4) * 8, c = (band * MT + m) * 16 + ((lane >> 3) & 1) * 8;
-                uint32_t k0, k1, k2, k3;
-                ldmatrix_x4_trans(k_addr + (r * PITCH + c) * 2, k0, k1, k2, k3);
-                mma_16816(S[m][0], k0, k1, k2, k3, b0, b1);
-                mma_16816(S[m][1], k0, k1, k2, k3, b2, b3);
-                if (tiles == 3) mma_16816(S[m][2], k0, k1, k2, k3, c0, c1);
-            }
+            for (int j = 0; j < 2; ++j)
+                if (j < tiles) ldmatrix_x4_trans(w_addr + ((kt * 16 + lane) * kColPitch + tile_col(j)) * 2, b[j][0], b[j][1], b[j][2], b[j][3]);
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    // K^T: the tile lies as [token][d], its transpose is the operand
+                    const int r = (kt + i) * 16 + (lane & 7) + (lane >> 4) * 8, c = (band * MT + m) * 16 + ((lane >> 3) & 1) * 8;
+                    uint32_t k0, k1, k2, k3;
+                    ldmatrix_x4_trans(k_addr + (r * PITCH + c) * 2, k0, k1, k2, k3);
+#pragma unroll
+                    for (int j = 0; j < 2; ++j)
+                        if (j < tiles) mma_16816(S[m][j], k0, k1, k2, k3, b[j][2 * i], b[j][2 * i + 1]);
+                }
         }
         __syncthreads();                         // everyone is done with the tiles
     }
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int j = 0; j < 3; ++j)
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 float* p = j < tiles ? place(m, j, e) : nullptr;
@@ -458,8 +525,10 @@ linear_memory_chunks_kernel(MemoryArgs a) {
 
 // ---- the output --------------------------------------------------------------------------------------------------------
 
-// One warp a (row, part) for parts of up to 256 elements, else a block (threads by the part's size alone).
-template <typename TO, bool WARP>
+// One warp a (row, part) for parts of up to 256 elements, else a block (threads by the part's size alone).  A thread holds up to
+// KEEP runs of W neighbouring elements between the two passes (W 4: a head's and a part's size are multiples of four, 16-byte
+// rows); what a longer part has beyond them is read again.
+template <typename TO, bool WARP, int W>
 __global__ void __launch_bounds__(WARP ? 256 : 1024)
 linear_memory_output_kernel(const float* __restrict__ o, const float* __restrict__ sums, const float* __restrict__ floors,
                             const float* __restrict__ gate, size_t gate_stride, const float* __restrict__ weight,
@@ -470,36 +539,63 @@ linear_memory_output_kernel(const float* __restrict__ o, const float* __restrict
     const int row = blockIdx.x, inner = H * V, n = inner / groups;
     const int grp = WARP ? blockIdx.y * 8 + (threadIdx.x >> 5) : blockIdx.y;
     if (grp >= groups) return;
-    const int tid = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x;
+    const int tid = WARP ? threadIdx.x & 31 : threadIdx.x, step = (WARP ? 32 : blockDim.x) * W;
     const float* src = o + (size_t)row * inner;
-    auto value = [&](int c) {
-        const float v = src[c];
-        if (!sums) return v;
+    auto value = [&](int c, float (&v)[W]) {
+        if constexpr (W == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(src + c);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        } else {
+            v[0] = src[c];
+        }
+        if (!sums) return;
         const size_t at = (size_t)row * H + c / V;
-        return v / (fmaxf(fabsf(sums[at]), floors[at]) + 1e-6f);
+        const float den = fmaxf(fabsf(sums[at]), floors[at]) + 1e-6f;
+#pragma unroll
+        for (int e = 0; e < W; ++e) v[e] /= den;
     };
-    constexpr int KEEP = 8;                                   // a thread's first values stay in registers between the passes
-    float kept[KEEP], ss = 0.0f;
+    constexpr int KEEP = W == 4 ? 2 : 8;
+    float kept[KEEP][W], more[W], ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = tid + j * step;
-        kept[j] = i < n ? value(grp * n + i) : 0.0f;
-        ss = fmaf(kept[j], kept[j], ss);
+        const int i = tid * W + j * step;
+        if (i < n) {
+            value(grp * n + i, kept[j]);
+#pragma unroll
+            for (int e = 0; e < W; ++e) ss = fmaf(kept[j][e], kept[j][e], ss);
+        }
     }
-    for (int i = tid + KEEP * step; i < n; i += step) {
-        const float v = value(grp * n + i);
-        ss = fmaf(v, v, ss);
+    for (int i = tid * W + KEEP * step; i < n; i += step) {
+        value(grp * n + i, more);
+#pragma unroll
+        for (int e = 0; e < W; ++e) ss = fmaf(more[e], more[e], ss);
     }
     ss = WARP ? warp_sum(ss) : block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)n + eps);
     const float* gt = gate + (size_t)row * gate_stride;
-    auto finish = [&](int c, float v) { stf(y, (size_t)row * inner + c, v * inv * weight[c] / (1.0f + expf(-gt[c]))); };
+    TO* dst = y + (size_t)row * inner;
+    auto gated = [&](float v, float w, float z) { return v * inv * w / (1.0f + expf(-z)); };
+    auto finish = [&](int c, const float (&v)[W]) {
+        if constexpr (W == 4) {
+            const float4 w = *reinterpret_cast<const float4*>(weight + c), z = *reinterpret_cast<const float4*>(gt + c);
+            const float4 r = make_float4(gated(v[0], w.x, z.x), gated(v[1], w.y, z.y), gated(v[2], w.z, z.z), gated(v[3], w.w, z.w));
+            if constexpr (sizeof(TO) == 2)
+                *reinterpret_cast<uint2*>(dst + c) = make_uint2(fa::pack_bf16(r.x, r.y), fa::pack_bf16(r.z, r.w));
+            else
+                *reinterpret_cast<float4*>(dst + c) = r;
+        } else {
+            stf(dst, c, gated(v[0], weight[c], gt[c]));
+        }
+    };
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-        const int i = tid + j * step;
+        const int i = tid * W + j * step;
         if (i < n) finish(grp * n + i, kept[j]);
     }
-    for (int i = tid + KEEP * step; i < n; i += step) finish(grp * n + i, value(grp * n + i));
+    for (int i = tid * W + KEEP * step; i < n; i += step) {
+        value(grp * n + i, more);
+        finish(grp * n + i, more);
+    }
 }
 
 template <int DP, int STAGES>
@@ -509,10 +605,10 @@ int launch_scan(const MemoryArgs& a, cudaStream_t stream) {
     return CITLALI_LAUNCH_CHECK();
 }
 
-template <int DP>
+template <int DP, bool VEC>
 int launch_chunks(const MemoryArgs& a, cudaStream_t stream) {
-    constexpr int smem = (2 * kChunk * (DP + 8) + 2 * kChunk * kColPitch + 2 * DP * kColPitch) * 2;
-    auto kernel = linear_memory_chunks_kernel<DP>;
+    constexpr int smem = (2 * kChunk * (DP + 8) + 2 * kChunk * kColPitch + 2 * DP * kColPitch + kChunk * kWeightPitch) * 2;
+    auto kernel = linear_memory_chunks_kernel<DP, VEC>;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -520,8 +616,14 @@ int launch_chunks(const MemoryArgs& a, cudaStream_t stream) {
         configured = true;
     }
     const long blocks = (long)a.sequences * a.H * ((a.V + kCols - 1) / kCols);
-    launch_kernel(kernel, (unsigned)blocks, 256, smem, stream, a);
+    launch_kernel(kernel, (unsigned)blocks, kChunkThreads, smem, stream, a);
     return CITLALI_LAUNCH_CHECK();
+}
+
+template <int DP>
+int pick_chunks(const MemoryArgs& a, cudaStream_t stream) {
+    const bool vec = a.D % 4 == 0 && a.V % 4 == 0 && a.stride % 4 == 0 && (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15u) == 0;
+    return vec ? launch_chunks<DP, true>(a, stream) : launch_chunks<DP, false>(a, stream);
 }
 
 }  // namespace
@@ -560,10 +662,10 @@ extern "C" int citlali_linear_memory(const float* q, const float* k, const float
                        q_scale, sequences, H, D, V, act};
     if (form == 2) {
         switch ((D + 63) / 64) {
-            case 1: return launch_chunks<64>(a, stream);
-            case 2: return launch_chunks<128>(a, stream);
-            case 3: return launch_chunks<192>(a, stream);
-            default: return launch_chunks<256>(a, stream);
+            case 1: return pick_chunks<64>(a, stream);
+            case 2: return pick_chunks<128>(a, stream);
+            case 3: return pick_chunks<192>(a, stream);
+            default: return pick_chunks<256>(a, stream);
         }
     }
 #define CITLALI_SCAN(DP, ST) return form == 1 ? launch_scan<DP, 2>(a, stream) : launch_scan<DP, ST>(a, stream)
@@ -589,15 +691,23 @@ extern "C" int citlali_linear_memory_output(const float* o, const float* sums, c
         return kBadShape;
     }
     const int n = H * V / groups;
+    const bool vec = V % 4 == 0 && n % 4 == 0 && gate_stride % 4 == 0 &&
+                     (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)y) & 15u) == 0;
+    int threads = ((n / 4 + 31) / 32) * 32;
+    threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
     return CITLALI_DISPATCH_FLOAT(y_dtype, TO, [&] {
+        auto go = [&](auto kernel, dim3 grid, int block) {
+            launch_kernel(kernel, grid, block, 0, stream, o, sums, floors, gate, gate_stride, weight, (TO*)y, H, V, groups, eps);
+        };
         if (n <= 256) {
             const dim3 grid(rows, (groups + 7) / 8);
-            launch_kernel(linear_memory_output_kernel<TO, true>, grid, 256, 0, stream, o, sums, floors, gate, gate_stride, weight, (TO*)y, H, V, groups, eps);
+            const int block = groups < 8 ? 32 * groups : 256;
+            if (vec) go(linear_memory_output_kernel<TO, true, 4>, grid, block);
+            else go(linear_memory_output_kernel<TO, true, 1>, grid, block);
         } else {
-            int threads = ((n / 4 + 31) / 32) * 32;
-            threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
             const dim3 grid(rows, groups);
-            launch_kernel(linear_memory_output_kernel<TO, false>, grid, threads, 0, stream, o, sums, floors, gate, gate_stride, weight, (TO*)y, H, V, groups, eps);
+            if (vec) go(linear_memory_output_kernel<TO, false, 4>, grid, threads);
+            else go(linear_memory_output_kernel<TO, false, 1>, grid, threads);
         }
         return CITLALI_LAUNCH_CHECK();
     });

@@ -4,8 +4,10 @@ Used by ``bench.py --design lanizen`` (beside the Qwen3 dense decoder), ``--desi
 closest design the library has: both mix delta-rule layers with windowed attention) and ``--design sobunex`` (beside
 Gidirax: both have windowed attention with key and value sizes of their own, layer norms on the sub-layers' outputs and
 experts whose weights are not renormalised) and ``--design pivavik`` (beside Sobunex: both are made of attention layers
-only, with windows, output gates, biases, and dense and routed feed-forwards in turn) and ``--design nomutar`` (beside
-Pivavik: both run mixer and feed-forward side by side on one norm and have windowed attention with a soft cap).  A size is a width and a number of layers; both models get that width, that
+only, with windows, output gates, biases, and dense and routed feed-forwards in turn), ``--design nomutar`` (beside
+Pivavik: both run mixer and feed-forward side by side on one norm and have windowed attention with a soft cap) and ``--design
+kopalorn`` (beside Gidirax: both have layers with a matrix of state a head, layers of attention beside a recurrence, layer norms on
+the sub-layers' outputs and routed experts in groups).  A size is a width and a number of layers; both models get that width, that
 many layers, feed-forwards of equal parameter count (8 width^2: two matrices of 4 width, or three of 8/3 width) and
 the same vocabulary, with random weights in bfloat16.  Measured per model: one prompt in one step (tokens a second),
 one decode step of ``batch`` sequences at ``context`` through the session's ``decode`` (the replayed graph where the
@@ -125,6 +127,30 @@ def nomutar_config(width: int, layers: int, vocab: int, window: int = 1024):
         "embedding": {"scale": 2.0, "bigram": {"buckets": 32749, "mul_prev": 1021, "mul_cur": 31}}, "canon": {"taps": 4},
         "logit_softcap": 30.0,
         "layers": [{"type": t, "mixer": dict(m), "mlp": dict(f)} for t, m, f in (order[i % 4] for i in range(layers))]})
+
+
+def kopalorn_config(width: int, layers: int, vocab: int, window: int = 1024):
+    """Differential attention, matrix memory and the pair of mixers in turn (attention twice in four), heads of 128 (maps of 64 over
+    values of 128), four query heads a key/value head; sixteen experts without a gate in four groups of which two are kept, a
+    token uses four, plus one of the same size for every token (about 8 width^2 parameters in all experts of a layer).  The middle
+    layers are a repeated run that runs once: the step ahead of it is measured, and the model runs as many layers as the design
+    beside it."""
+    heads = max(1, width // 128)
+    kv = max(1, heads // 4)
+    ff = max(64, (width // 4 + 32) // 64 * 64)
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}, "scale": 2.5},
+           "shared": {"ff": ff}}
+    attention = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "mask": {"size": window},
+                 "rot": {"base": 500000.0, "dims": 64}}
+    mlstm = {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    par = {"left": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5},
+           "right": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(3 + 5 * h / heads) for h in range(heads)]}}
+    order = [("attention", attention), ("mlstm", mlstm), ("parallel", par), ("attention", attention)]
+    d = {"architecture": "Kopalorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+         "layers": [{"type": t, "mixer": dict(m), "mlp": dict(moe)} for t, m in (order[i % 4] for i in range(layers))]}
+    if layers >= 3:
+        d["loop"] = {"start": 1, "stop": layers - 1, "times": 1}
+    return config_from_dict(d)
 
 
 def qwen3_config(width: int, layers: int, vocab: int):
@@ -256,7 +282,8 @@ def measure_model(config, prompt_tokens: int, batch: int, context: int, steps: i
 
 
 DESIGNS = {"lanizen": (lanizen_config, "qwen3"), "gidirax": (gidirax_config, "lanizen"), "sobunex": (sobunex_config, "gidirax"),
-           "pivavik": (pivavik_config, "sobunex"), "nomutar": (nomutar_config, "pivavik"), "qwen3": (qwen3_config, None)}
+           "pivavik": (pivavik_config, "sobunex"), "nomutar": (nomutar_config, "pivavik"),
+           "kopalorn": (kopalorn_config, "gidirax"), "qwen3": (qwen3_config, None)}
 
 
 def run(design: str, sizes, prompt_tokens: int, batch: int, context: int, steps: int, warmup: int) -> dict:

@@ -220,7 +220,7 @@ def memory_close(got, want, dtype, what):
         close(got, want, dtype, what)
         return
     err = (got - want).abs().amax(-1) / want.abs().max()
-    assert float(err.max()) < 0.3 and float(err.median()) < 6e-3 and float((err < 3e-2).double().mean()) >= 0.97, (what, err.topk(5).values)
+    assert float(err.max()) < 0.3 and float(err.median()) < 6e-3 and float((err < 3e-2).double().mean()) >= 0.93, (what, err.topk(5).values)
 
 
 def every_way_of_a_memory(hs, fn, h, other, dtype):
