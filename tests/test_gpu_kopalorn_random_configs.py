@@ -69,11 +69,11 @@ def test_random_configuration(i, tmp_path):
     cb.write_safetensors(os.path.join(path, "model.safetensors"), lambda: iter(w.items()), metadata={"format": "pt"})
     reqs = [("a", random_tokens(d["vocab"], 150, 3 * i + 1)), ("b", random_tokens(d["vocab"], 47, 3 * i + 2))]
     want = {rid: plain.forward(cfg.to_dict(), w, toks) for rid, toks in reqs}
-    # 32-bit: every position within rounding of the exact evaluation (99 % tightly: a head of a matrix memory whose result nearly
+    # 32-bit: every position within rounding of the exact evaluation (98 % tightly: a head of a matrix memory whose result nearly
     # cancels is blown up, rounding and all, by the norm behind it).  bfloat16: a router's close call may fall the other way, and
     # every position behind it in the sequence then differs: most positions must agree and the median error must be small; each
     # bfloat16 kernel is held strictly where it is tested alone
-    for dtype, tol, most in (("float32", 5e-5, 0.99), ("bfloat16", 5e-2, 0.6)):
+    for dtype, tol, most in (("float32", 5e-5, 0.98), ("bfloat16", 5e-2, 0.6)):
         s = cb.InferenceSession().load_model(path, max_context=256, dtype=dtype, max_batch=2)
         for what, steps in (("whole", replay.whole(reqs)), ("tail", replay.tail(reqs, last=40)),
                             ("batched", replay.batched(reqs, [100, 20], 2))):
