@@ -234,7 +234,7 @@ struct DecodeOptions {
     const float* gate = nullptr;
     size_t gate_stride = 0;
     int turn_pairs = 0, dk = 0, dv = 0;
-    float* out32 = nullptr;            // the result in float32, rows out32_stride apart, instead of the rounded one
+    float* out32 = nullptr;            // the result in float32, rows out32_stride apart, instead of the rounded one (kExact false only)
     size_t out32_stride = 0;
 };
 
@@ -243,12 +243,17 @@ __device__ __forceinline__ float sink_share(const DecodeOptions& opt, int head, 
 }
 
 // The head's `dv` results value(i): turned back, gated, rounded, stored.
-template <typename Value>
+template <bool kWide, typename Value>
 __device__ __forceinline__ void store_head(const DecodeOptions& opt, int row, int head, int dv, __nv_bfloat16* out_head, int tid, Value value) {
+    if (kWide && opt.out32) {                // (not with turns)
+        float* wide = opt.out32 + (size_t)row * opt.out32_stride + (size_t)head * dv;
+        const float* z = opt.gate ? opt.gate + (size_t)row * opt.gate_stride + (size_t)head * dv : nullptr;
+        for (int i = tid; i < dv; i += 128) wide[i] = z ? value(i) / (1.0f + expf(-z[i])) : value(i);
+        return;
+    }
     auto store = [&](int i, float r) {
         if (opt.gate) r *= 1.0f / (1.0f + expf(-opt.gate[(size_t)row * opt.gate_stride + (size_t)head * dv + i]));
-        if (opt.out32) opt.out32[(size_t)row * opt.out32_stride + (size_t)head * dv + i] = r;
-        else out_head[i] = __float2bfloat16_rn(r);
+        out_head[i] = __float2bfloat16_rn(r);
     };
     if (opt.turns) {
         const int half = dv / 2;
@@ -266,7 +271,7 @@ __device__ __forceinline__ void store_head(const DecodeOptions& opt, int row, in
 
 // One head's (m, l, O) of `runs` consecutive runs of its keys ([run][D + 2] at `base`, m in log2 units), merged in run
 // order into the head's output.  kFromL2: the runs were written by other blocks to global memory (read past L1).
-template <int kBlocks, int D, bool kFromL2>
+template <int kBlocks, int D, bool kFromL2, bool kWide>
 __device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfloat16* out_head, int tid, const DecodeOptions& opt,
                                            int row, int head, int dv) {
     auto at = [&](size_t i) { return kFromL2 ? __ldcg(base + i) : base[i]; };
@@ -287,7 +292,7 @@ __device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfl
         wz[z] = f;
     }
     const float inv = 1.0f / L;
-    store_head(opt, row, head, dv, out_head, tid, [&](int i) {
+    store_head<kWide>(opt, row, head, dv, out_head, tid, [&](int i) {
         float a = 0.0f;
 #pragma unroll
         for (int z = 0; z < kBlocks; ++z)
@@ -298,11 +303,11 @@ __device__ __forceinline__ void merge_runs(const float* base, int runs, __nv_bfl
 
 // Block `rank` of a cluster merges heads rank, rank + split, ... over the (m, l, O) of all blocks' runs, which
 // they have sent to `gathered` ([head / split][sender][D + 2]), in rank order.
-template <int kBlocks, int D>
+template <int kBlocks, int D, bool kWide>
 __device__ __forceinline__ void merge_gathered_heads(const float* gathered, __nv_bfloat16* out_row, int rank, int split, int heads_here, int tid,
                                                      const DecodeOptions& opt, int row, int head0, int dv) {
     for (int h = rank; h < heads_here; h += split)
-        merge_runs<kBlocks, D, false>(gathered + (size_t)((h / split) * split) * (D + 2), split, out_row + (size_t)h * dv, tid, opt, row,
+        merge_runs<kBlocks, D, false, kWide>(gathered + (size_t)((h / split) * split) * (D + 2), split, out_row + (size_t)h * dv, tid, opt, row,
                                       head0 + h, dv);
 }
 
@@ -608,7 +613,7 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         for (int h = 0; h < heads_here; ++h) {
             const float* mine = gathered + h * (D + 2);
             const float inv = 1.0f / (mine[1] + sink_share(opt, head0 + h, mine[0]));
-            store_head(opt, row, head0 + h, dv, out_row + (size_t)h * dv, tid, [&](int i) { return mine[2 + i] * inv; });
+            store_head<!kExact>(opt, row, head0 + h, dv, out_row + (size_t)h * dv, tid, [&](int i) { return mine[2 + i] * inv; });
         }
         return;
     }
@@ -632,7 +637,7 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         if (!counted_last) return;
         __threadfence();
         for (int h = 0; h < heads_here; ++h)
-            merge_runs<kMaxRunsByLength, D, true>(partial + ((size_t)row * nq + head0 + h) * chunks * (D + 2), split,
+            merge_runs<kMaxRunsByLength, D, true, !kExact>(partial + ((size_t)row * nq + head0 + h) * chunks * (D + 2), split,
                                                   out_row + (size_t)h * dv, tid, opt, row, head0 + h, dv);
         return;
     }
@@ -649,10 +654,10 @@ attention_decode_tc_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     }
     cluster_arrive();
     cluster_wait();
-    if (split <= 2) merge_gathered_heads<2, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
-    else if (split <= 4) merge_gathered_heads<4, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
-    else if (split <= 8) merge_gathered_heads<8, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
-    else merge_gathered_heads<kMaxClusterBlocks, D>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    if (split <= 2) merge_gathered_heads<2, D, !kExact>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else if (split <= 4) merge_gathered_heads<4, D, !kExact>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else if (split <= 8) merge_gathered_heads<8, D, !kExact>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
+    else merge_gathered_heads<kMaxClusterBlocks, D, !kExact>(gathered, out_row, rank, split, heads_here, tid, opt, row, head0, dv);
 }
 
 static int g_forced_split = 0;     // > 0: blocks per (sequence, head group), for tuning
@@ -901,6 +906,10 @@ extern "C" int citlali_attention_decode_with(const void* q, int q_stride, const 
                        "pages of 64)", head_dim, value_dim, page_size);
         return kBadShape;
     }
+    if (out32 != nullptr && turns != nullptr) {
+        set_last_error("attention_decode_with: an output that is turned back is not left in float32");
+        return kBadShape;
+    }
     if (q_stride % 8 != 0 || ((uintptr_t)q & 15u) || ((uintptr_t)turns & 7u)) {
         set_last_error("attention_decode_with: query rows must be 16-byte aligned (row pitch %d elements)", q_stride);
         return kBadAlignment;
@@ -920,7 +929,7 @@ extern "C" int citlali_attention_decode_with(const void* q, int q_stride, const 
 #define CITLALI_TC(DD, EX) return launch_tc<DD, EX>(q, q_stride, k_pool, v_pool, page_table, page_table_stride, row_slot, row_pos, \
                                                       out, out_stride, rows, nq, nkv, window, scale, opt, stream, partial, \
                                                       partial_floats, counters, counter_ints)
-    if (head_dim == value_dim) {
+    if (head_dim == value_dim && out32 == nullptr) {
         switch (head_dim) {
             case 16: CITLALI_TC(16, true);
             case 32: CITLALI_TC(32, true);
