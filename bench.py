@@ -328,7 +328,7 @@ class ClockSampler:
 def run_design(args):
     """``--design``: a design beside another of the library's at equal width and depth (Lanizen beside the Qwen3 decoder,
     Gidirax beside Lanizen, Sobunex beside Gidirax, Pivavik beside Sobunex,
-    Nomutar beside Pivavik; see ``citlali_b200.measure``).  One JSON line; the default workload and its line are not touched."""
+    Nomutar beside Pivavik, Kopalorn beside Gidirax; see ``citlali_b200.measure``).  One JSON line; the default workload and its line are not touched."""
     import citlali_b200  # noqa: F401  (loads the package under its importable name)
     from citlali_b200 import measure
     sizes = [s for s in args.sizes.split(",") if s]
